@@ -101,6 +101,22 @@ class LayerCache:
                 v[t // S2 - page0, :, :, t % S2, :] = values[lo - t0:hi - t0]
             page0 += n
 
+    def reserve(self, steps):
+        """Room for `steps` more tokens of the sequences already cached."""
+        B, nkv, hd = self.dims()
+        self.ensure(B, nkv, hd, steps, self.arenas[0][0].dtype, self.arenas[0][0].device)
+
+    def fits(self, batch, need):
+        """Whether a new request of `batch` sequences and `need` tokens can use this storage from its first page on."""
+        return bool(self.arenas) and self.contiguous() and self.dims()[0] == batch and self.capacity() >= need
+
+    def reset(self):
+        self.offset = 0
+
+    def storage_key(self):
+        """Changes when the device memory behind the cache does (a recorded decode step holds its addresses)."""
+        return [id(a[0]) for a in self.arenas]
+
     def select_batch(self, idx, repeat=1):
         new = []
         for k, v in self.arenas:
@@ -111,15 +127,122 @@ class LayerCache:
         self._rebuild_tables()
 
 
+class HybridLayerCache:
+    """What a layer of a hybrid decoder keeps per sequence: latent rows in 32-token pages (latent attention) and named
+    32-bit state tensors [B, ...] that every token updates in place (convolution inputs, the matrix state of a recurrence).
+
+    Pages are [B, 32, R] slabs reached through a device array of addresses, as in LayerCache. With a sliding window only
+    the last `window` tokens are ever read: the page table stops growing at the number of pages a window can touch, and
+    token t then lives in page (t // 32) mod pages, i.e. old pages are used again. While the table still grows no page index
+    has wrapped, so growth moves nothing."""
+
+    def __init__(self):
+        self.arenas = []     # tensors [pages, B, 32, R]
+        self.ptrs = None     # int64 [pages]
+        self.window = 0      # tokens ever looked back at, 0: all
+        self.states = {}
+        self.offset = 0
+        self.live = None     # rows of the running multi-token call [B, L, R], for the layers that share them
+
+    def pages(self):
+        return sum(a.shape[0] for a in self.arenas)
+
+    def capacity(self):
+        n = self.pages()
+        return (1 << 30) if not self.arenas or (self.window and n >= self.window_pages()) else n * S2
+
+    def window_pages(self):
+        """Pages that `window` consecutive tokens can touch."""
+        return (self.window + S2 - 2) // S2 + 1
+
+    def batch(self):
+        for t in self.states.values():
+            return t.shape[0]
+        return self.arenas[0].shape[1] if self.arenas else None
+
+    def ensure_latent(self, B, R, tokens, window, dtype, device):
+        """Pages for the tokens up to index offset + tokens - 1."""
+        if self.arenas and tuple(self.arenas[0].shape[1:]) != (B, S2, R):
+            raise _lib.TpxError("latent cache shape changed between calls")
+        self.window = window
+        need = (self.offset + tokens + S2 - 1) // S2
+        if need > self.pages():
+            need += KV_CACHE_INC_SIZE // S2
+        if window:
+            need = min(need, self.window_pages())
+        if need > self.pages():
+            self.arenas.append(torch.zeros((need - self.pages(), B, S2, R), dtype=dtype, device=device))
+            self._rebuild_table()
+
+    def _rebuild_table(self):
+        if not self.arenas:
+            return
+        addrs = []
+        for a in self.arenas:
+            step = a.stride(0) * a.element_size()
+            addrs += [a.data_ptr() + i * step for i in range(a.shape[0])]
+        self.ptrs = torch.tensor(addrs, dtype=torch.int64, device=self.arenas[0].device)
+
+    def state(self, name, shape, device):
+        """The named state, zero when a sequence starts."""
+        t = self.states.get(name)
+        if t is None:
+            t = self.states[name] = torch.zeros(shape, dtype=torch.float32, device=device)
+        elif tuple(t.shape) != tuple(shape):
+            raise _lib.TpxError(f"state '{name}' changed shape between calls")
+        return t
+
+    def reserve(self, steps):
+        if self.arenas:
+            a = self.arenas[0]
+            self.ensure_latent(a.shape[1], a.shape[3], steps, self.window, a.dtype, a.device)
+
+    def fits(self, batch, need):
+        return self.batch() == batch and self.capacity() >= need
+
+    def reset(self):
+        self.offset, self.live = 0, None
+        for t in self.states.values():
+            t.zero_()
+
+    def storage_key(self):
+        return [t.data_ptr() for t in self.arenas + list(self.states.values())]
+
+    def dims(self):
+        return (self.batch(),)
+
+    def crop(self, max_length):
+        if max_length == 0:
+            self.reset()
+        elif max_length < self.offset:
+            raise _lib.TpxError("a recurrent state cannot be rolled back to an earlier token")
+
+    def select_batch(self, idx, repeat=1):
+        def pick(t, dim):
+            if repeat > 1:
+                t = t.repeat_interleave(repeat, dim=dim)
+            return t.index_select(dim, idx.to(t.device)).contiguous()
+        self.arenas = [pick(a, 1) for a in self.arenas]
+        self.states = {n: pick(t, 0) for n, t in self.states.items()}
+        self._rebuild_table()
+
+
 class TppCache:
     """torch.classes.tpp_llm.TppCache (src/csrc/llm/attn.h:229-404)."""
 
     def __init__(self):
         self.layers = []
+        self.start = None  # int32 [B]: leading padding per sequence, kept by models whose state depends on it
 
     def layer(self, idx):
         while len(self.layers) <= idx:
             self.layers.append(LayerCache())
+        return self.layers[idx]
+
+    def hybrid_layer(self, idx):
+        """Layer idx of a model whose layers keep latent pages and recurrent states instead of keys and values."""
+        while len(self.layers) <= idx:
+            self.layers.append(HybridLayerCache())
         return self.layers[idx]
 
     def update(self, key_states, value_states, layer_idx):
@@ -159,8 +282,25 @@ class TppCache:
 
     def crop(self, max_length):
         for lc in self.layers:
-            if lc.offset > max_length:
+            if isinstance(lc, HybridLayerCache):
+                lc.crop(max_length)
+            elif lc.offset > max_length:
                 lc.offset = max_length
+
+    def reset(self):
+        """Forget every sequence; the storage stays."""
+        self.start = None
+        for lc in self.layers:
+            lc.reset()
+
+    def keep_sequences(self, rows):
+        """Only the sequences `rows` (in that order) go on; what the others held is given back to the allocator."""
+        for lc in self.layers:
+            dev = next((t.device for t in list(getattr(lc, "states", {}).values()) + [a[0] for a in lc.arenas]), None)
+            if dev is not None:
+                lc.select_batch(torch.as_tensor(rows, dtype=torch.long, device=dev))
+        if self.start is not None:
+            self.start = self.start.index_select(0, torch.as_tensor(rows, dtype=torch.long, device=self.start.device))
 
     def reorder_cache(self, beam_idx):
         """TppCache::reorder_cache (src/csrc/llm/attn.h:327-403): after the call, sequence i continues the history
@@ -170,8 +310,11 @@ class TppCache:
         indices is first repeated per beam, as the reference does (attn.h:345-367)."""
         beam_idx = beam_idx.to(torch.long)
         B = beam_idx.shape[0]
+        if self.start is not None:
+            s = self.start.repeat_interleave(B // self.start.shape[0])
+            self.start = s.index_select(0, beam_idx.to(s.device))
         for lc in self.layers:
-            if not lc.arenas:
+            if not lc.arenas and not getattr(lc, "states", None):
                 continue
             CB = lc.dims()[0]
             rep = 1
@@ -179,7 +322,7 @@ class TppCache:
                 if B % CB != 0:
                     raise _lib.TpxError(f"New batch ({B}) must be multiple of cached batch size ({CB})")
                 rep = B // CB
-            lc.select_batch(beam_idx.to(lc.arenas[0][0].device), rep)
+            lc.select_batch(beam_idx.to(lc.arenas[0][0].device) if lc.arenas else beam_idx, rep)
 
 
 def attention(q, kc, vc, mask, key_len, causal=True, out_bsnrh=False, dev_len=None, pages=None):

@@ -68,6 +68,16 @@ _SIGS = {
     "tpx_attention": (c_int, [c_vp, c_vp, c_vp, c_vp] + [c_i64] * 7 + [c_int, c_int, c_vp, c_vp, c_vp, c_sz, c_vp]),
     "tpx_attention_tc_status": (c_int, [c_vp, ctypes.POINTER(ctypes.c_uint)]),
     "tpx_align_and_invert_mask": (c_int, [c_vp, c_i64, c_i64, c_i64, ctypes.c_uint16, c_vp, c_vp]),
+    "tpx_linear": (c_int, [c_vp, c_vp]),
+    "tpx_postnorm_conv": (c_int, [c_vp, c_vp]),
+    "tpx_postnorm_final": (c_int, [c_vp, c_vp]),
+    "tpx_argmax_f32": (c_int, [c_vp, c_i64, c_i64, c_vp, c_vp]),
+    "tpx_latent_prep": (c_int, [c_vp, c_vp]),
+    "tpx_latent_gather": (c_int, [c_vp] + [c_i64] * 6 + [c_vp, c_int, c_vp]),
+    "tpx_latent_absorb": (c_int, [c_vp, c_vp]),
+    "tpx_latent_attn": (c_int, [c_vp, c_vp]),
+    "tpx_latent_value": (c_int, [c_vp, c_vp]),
+    "tpx_delta_rule": (c_int, [c_vp, c_vp]),
     "tpx_qlinear": (c_int, [c_int, c_vp, c_vp, c_vp, c_vp, c_i64, c_vp, c_i64, c_i64, c_i64, c_vp, c_int, c_vp, c_vp,
                             c_f32, c_vp, c_vp, c_sz, c_vp]),
 }
@@ -75,6 +85,15 @@ _SIGS = {
 
 class TpxError(RuntimeError):
     pass
+
+
+def use_library(path):
+    """Load the library from `path` (a build of only some components); before the first kernel call."""
+    global _SO
+    if _lib is not None and path != _SO:
+        raise TpxError("the CUDA library is already loaded")
+    if not os.environ.get("TPX_LIBRARY"):
+        _SO = path
 
 
 def lib():
@@ -108,6 +127,25 @@ class LlamaLayerIOStruct(ctypes.Structure):
                                                  "inter", "out", "scratch")] + \
                [("scratch_bytes", ctypes.c_size_t), ("attn_scratch", ctypes.c_void_p), ("attn_scratch_bytes", ctypes.c_size_t),
                 ("handoff", ctypes.c_void_p), ("handoff_bytes", ctypes.c_size_t)]
+
+
+def _struct(name, **groups):
+    """A ctypes mirror of a parameter block of include/tpx_hybrid.h: group name = field type, value = its fields in order;
+    a digit behind the type name only keeps the keywords distinct."""
+    types = {"p": ctypes.c_void_p, "l": ctypes.c_int64, "f": ctypes.c_float, "i": ctypes.c_int, "z": ctypes.c_size_t}
+    return type(name, (ctypes.Structure,), {"_fields_": [(n, types[g[0]]) for g, names in groups.items() for n in names.split()]})
+
+
+LinearStruct = _struct("LinearStruct", p="w x bias act_params y", l="M N K ldw ldx ldy", i="f32 out_f32 act act_from", p2="scratch", z="scratch_bytes")
+PostnormConvStruct = _struct("PostnormConvStruct", p="ids embed x y w conv state start dev_len x_out h", l="B S D ldh past", f="alpha eps", i="taps f32")
+PostnormFinalStruct = _struct("PostnormFinalStruct", p="x y w w_final rows out", l="n D ldo", f="alpha eps", i="f32")
+LatentPrepStruct = _struct("LatentPrepStruct", p="proj q_norm kv_norm freq start dev_len cq cos_sin gate lat pages",
+                           l="B S L ldp ldq past npages q_rank kv_rank krp rot_dim R heads", f="eps", i="own_kv f32")
+LatentAbsorbStruct = _struct("LatentAbsorbStruct", p="q w_uk cos_sin qa", l="T ldq heads dim kv_rank krp rot_dim R", i="f32")
+LatentAttnStruct = _struct("LatentAttnStruct", p="qa lat pages start dev_len ol", l="B S L past npages heads krp R window", f="scale", i="f32",
+                           p2="scratch", z="scratch_bytes")
+LatentValueStruct = _struct("LatentValueStruct", p="ol gate w_uv out", l="T heads vdim krp ldo", i="f32")
+DeltaRuleStruct = _struct("DeltaRuleStruct", p="proj wraw a_bias norm_w start dev_len state raw out", l="B S past ldp ldo heads dim", f="eps", i="f32")
 
 
 def check(rc):
@@ -168,7 +206,7 @@ def assert_no_kernel_error(sync=True):
         code = inst.error_code()
         if code:
             raise TpxError(f"the peer-memory all-reduce gave up waiting for rank {code - 1}")
-    if _lib is not None and torch.cuda.is_available():
+    if _lib is not None and hasattr(_lib, "tpx_attention_tc_status") and torch.cuda.is_available():
         st = ctypes.c_uint(0)
         check(_lib.tpx_attention_tc_status(stream(), ctypes.byref(st)))
         if st.value:

@@ -17,15 +17,50 @@
 // One CTA per SM walks a contiguous range of output tiles (the token tiles of one feature tile are neighbours, so a
 // weight tile fetched for the first of them is found in L2 by the others). Two accumulators in tensor memory: the
 // epilogue of a tile runs under the MMAs of the next. At decode sizes the kernel is a plain stream of W at HBM rate.
+#include "tpx_hybrid.cuh"
 #include "tpx_tc_ptx.cuh"
 
 namespace tpx {
+
+// Epilogue of tpx_linear: fp32 bias, row stride, fp32 or bf16 result, activation from a column on.
+struct BfEx {
+  const float *bias, *ap;
+  void* y;
+  long long ldy;
+  int on, out_f32, act, act_from;
+};
 
 struct BfParams {
   TcParams t;   // epilogue fields (bias, act, mul_in, res, res_scale, y, M, N, err)
   int ksteps;   // k steps of 64 (K rounded up)
   int TN, TM;   // feature tiles, token tiles
+  BfEx ex;
 };
+
+// 16 consecutive tokens of output feature n; the lanes of a warp hold 32 neighbouring features
+__device__ __forceinline__ void bf_finish16_ex(const BfEx& e, int M, int tok0, int n, const float (&v)[16]) {
+  const int live = M - tok0;
+  const float b = e.bias ? e.bias[n] : 0.0f;
+  float x[16];
+#pragma unroll
+  for (int j = 0; j < 16; j++) x[j] = v[j] + b;
+  if (e.act && n >= e.act_from) {
+    const float a0 = e.ap ? e.ap[0] : 0.0f, a1 = e.ap ? e.ap[1] : 0.0f;
+#pragma unroll
+    for (int j = 0; j < 16; j++) x[j] = hy_act(x[j], e.act, a0, a1);
+  }
+  if (e.out_f32) {
+    float* y = reinterpret_cast<float*>(e.y) + (long long)tok0 * e.ldy + n;
+#pragma unroll
+    for (int j = 0; j < 16; j++)
+      if (j < live) y[j * e.ldy] = x[j];
+  } else {
+    uint16_t* y = reinterpret_cast<uint16_t*>(e.y) + (long long)tok0 * e.ldy + n;
+#pragma unroll
+    for (int j = 0; j < 16; j++)
+      if (j < live) y[j * e.ldy] = f32_to_bf16_bits(x[j]);
+  }
+}
 
 template <int TOK>
 struct BfCfg {
@@ -176,7 +211,10 @@ linear_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
         for (int j = 0; j < 16; j++) { v[j] = __uint_as_float(a[j]); v2[j] = 0.0f; }
-        if (n < p.t.N && tok0 + c0 < p.t.M) tc_finish16<false>(p.t, tok0 + c0, n, v, v2);
+        if (n < p.t.N && tok0 + c0 < p.t.M) {
+          if (p.ex.on) bf_finish16_ex(p.ex, p.t.M, tok0 + c0, n, v);
+          else tc_finish16<false>(p.t, tok0 + c0, n, v, v2);
+        }
       }
       tc_fence_before();
       __syncwarp();
@@ -191,8 +229,8 @@ linear_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
   }
 }
 
-// 2-D bf16 tensor [rows][cols] (row stride cols * 2 bytes), box = 64 columns x box_rows, 128-byte swizzle.
-static int bf_make_map(CUtensorMap* m, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows) {
+// 2-D bf16 tensor [rows][cols] (row stride ld elements), box = 64 columns x box_rows, 128-byte swizzle.
+static int bf_make_map(CUtensorMap* m, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows) {
   typedef CUresult (*Fn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
                          const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
   static Fn fn = nullptr;
@@ -205,7 +243,7 @@ static int bf_make_map(CUtensorMap* m, const void* base, uint64_t rows, uint64_t
   }
   TPX_REQUIRE(fn, TPX_ERR_CUDA, "cuTensorMapEncodeTiled is not available from this driver");
   cuuint64_t gdim[2] = {cols, rows};
-  cuuint64_t gstr[1] = {cols * 2};
+  cuuint64_t gstr[1] = {ld * 2};
   cuuint32_t box[2] = {64, box_rows};
   cuuint32_t estr[2] = {1, 1};
   CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), gdim, gstr, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
@@ -231,6 +269,39 @@ static int bf_launch(const CUtensorMap& w, const CUtensorMap& x, const BfParams&
   return TPX_OK;
 }
 
+// Tiles, tensor maps and launch for a filled epilogue.
+static int bf_run(BfParams& p, const void* w, const void* x, int64_t M, int64_t N, int64_t K, int64_t ldw, int64_t ldx, cudaStream_t st) {
+  const int tok = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
+  p.t.M = (int)M; p.t.N = (int)N; p.t.K = (int)K;
+  p.ksteps = (int)((K + 63) / 64);
+  p.TN = (int)((N + 127) / 128);
+  p.TM = (int)((M + tok - 1) / tok);
+  CUtensorMap mw, mx;
+  int rc = bf_make_map(&mw, w, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, 128);
+  if (rc) return rc;
+  rc = bf_make_map(&mx, x, (uint64_t)M, (uint64_t)K, (uint64_t)ldx, (uint32_t)tok);
+  if (rc) return rc;
+  switch (tok) {
+    case 16: return bf_launch<16>(mw, mx, p, st);
+    case 32: return bf_launch<32>(mw, mx, p, st);
+    case 64: return bf_launch<64>(mw, mx, p, st);
+    case 128: return bf_launch<128>(mw, mx, p, st);
+    default: return bf_launch<256>(mw, mx, p, st);
+  }
+}
+
+int linear_tc_ex(const TpxLinear& a, cudaStream_t st) {
+  TPX_REQUIRE(a.K % 8 == 0 && a.ldx % 8 == 0 && a.ldw % 8 == 0, TPX_ERR_ARG, "linear: bf16 rows must be whole 16-byte units (K=%ld ldx=%ld ldw=%ld)",
+              (long)a.K, (long)a.ldx, (long)a.ldw);
+  TPX_REQUIRE((((uintptr_t)a.w | (uintptr_t)a.x) & 15) == 0 && ((uintptr_t)a.scratch & 255) == 0, TPX_ERR_ARG, "linear: misaligned pointer");
+  TPX_REQUIRE(a.scratch && a.scratch_bytes >= kTcCounterBytes, TPX_ERR_SCRATCH, "linear: scratch of %zu bytes needed, %zu given", kTcCounterBytes,
+              a.scratch_bytes);
+  BfParams p = {};
+  p.t.err = reinterpret_cast<unsigned*>(reinterpret_cast<unsigned char*>(a.scratch) + kTcCounterBytes - 4);
+  p.ex = {a.bias, a.act_params, a.y, (long long)a.ldy, 1, a.out_f32, a.act, a.act_from};
+  return bf_run(p, a.w, a.x, a.M, a.N, a.K, a.ldw, a.ldx, st);
+}
+
 }  // namespace tpx
 
 using namespace tpx;
@@ -252,25 +323,8 @@ extern "C" int tpx_linear_bf16_tc(const uint16_t* w, const uint16_t* x, int64_t 
   TPX_REQUIRE((((uintptr_t)w | (uintptr_t)x) & 15) == 0 && ((uintptr_t)scratch & 255) == 0, TPX_ERR_ARG, "linear_bf16_tc: misaligned pointer");
   TPX_REQUIRE(scratch && scratch_bytes >= kTcCounterBytes, TPX_ERR_SCRATCH, "linear_bf16_tc: scratch of %zu bytes needed, %zu given",
               kTcCounterBytes, scratch_bytes);
-  const int tok = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
   BfParams p = {};
   p.t.bias = bias; p.t.mul_in = mul_in; p.t.res = res; p.t.res_scale = res_scale; p.t.y = y; p.t.act = act;
-  p.t.M = (int)M; p.t.N = (int)N; p.t.K = (int)K;
   p.t.err = reinterpret_cast<unsigned*>(reinterpret_cast<unsigned char*>(scratch) + kTcCounterBytes - 4);
-  p.ksteps = (int)((K + 63) / 64);
-  p.TN = (int)((N + 127) / 128);
-  p.TM = (int)((M + tok - 1) / tok);
-  CUtensorMap mw, mx;
-  int rc = bf_make_map(&mw, w, (uint64_t)N, (uint64_t)K, 128);
-  if (rc) return rc;
-  rc = bf_make_map(&mx, x, (uint64_t)M, (uint64_t)K, (uint32_t)tok);
-  if (rc) return rc;
-  cudaStream_t st = (cudaStream_t)stream;
-  switch (tok) {
-    case 16: return bf_launch<16>(mw, mx, p, st);
-    case 32: return bf_launch<32>(mw, mx, p, st);
-    case 64: return bf_launch<64>(mw, mx, p, st);
-    case 128: return bf_launch<128>(mw, mx, p, st);
-    default: return bf_launch<256>(mw, mx, p, st);
-  }
+  return bf_run(p, w, x, M, N, K, K, K, (cudaStream_t)stream);
 }

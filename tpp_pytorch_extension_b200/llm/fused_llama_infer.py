@@ -89,11 +89,11 @@ class _DecodeSession:
 
     def cache_fits(self, batch, need):
         layers = self.cache.get_cpp().layers
-        return self.batch == batch and layers and all(lc.contiguous() and lc.capacity() >= need for lc in layers)
+        return self.batch == batch and layers and all(lc.fits(batch, need) for lc in layers)
 
     def graph_fits(self, cpp, cap):
         return (self.graph is not None and self.capacity == cap
-                and self.arenas == [id(a[0]) for lc in cpp.layers for a in lc.arenas])
+                and self.arenas == [k for lc in cpp.layers for k in lc.storage_key()])
 
 
 class LlamaRunner(torch.nn.Module):
@@ -107,6 +107,7 @@ class LlamaRunner(torch.nn.Module):
         # row-parallel followed by an all-reduce (fused_llama_infer.py:218-224)
         self.lm_head_w = lm_head_w
         self.only_last_logit = True
+        self.logit_rows = None  # int64 rows of the call's B * S tokens whose logits [rows, V] are wanted, instead of the above
 
     def _embed(self, ids, positions):
         """Token embedding; model families with learned position embeddings add them here."""
@@ -117,7 +118,9 @@ class LlamaRunner(torch.nn.Module):
 
     def _head(self, hs):
         """Final norm + lm_head on the last position (logits slicing of the reference, fused_llama_infer.py:385-390)."""
-        if self.only_last_logit:
+        if self.logit_rows is not None:
+            hs = hs.reshape(-1, hs.shape[-1])[self.logit_rows]
+        elif self.only_last_logit:
             hs = hs[:, -1:, :]
         hs = self._final_norm(hs)
         # lm_head_w is a bf16 matrix (the reference's default) or a quantized tensor (its --quantize-lm-head): both go
@@ -132,6 +135,21 @@ class LlamaRunner(torch.nn.Module):
         if logits.shape[-1] != self.shape.vocab_size:  # a quantized head padded to whole row groups
             logits = logits[..., :self.shape.vocab_size]
         return logits
+
+    def _pick(self, logits):
+        """Greedy token of the last position, [B, 1]."""
+        return fused_llm_cpp.argmax_rows(logits[:, -1]).unsqueeze(-1)
+
+    def _reserve(self, cpp, batch, tokens, device):
+        """Cache room for a request of known size, in one piece per layer."""
+        for i, layer in enumerate(self.layers):
+            cpp.layer(i).ensure(batch, layer.Nkv, layer.H, tokens, torch.bfloat16, device)
+
+    def _decode_mask(self, cpp, mask, past, cap):
+        """What the layers get as their mask during decoding: the keep-mask of the cached tokens, additive, up to the
+        cache's capacity (positions not yet written are excluded by the length, not by the mask)."""
+        ones = torch.ones((mask.shape[0], cap - past), dtype=torch.bfloat16, device=mask.device)
+        return cpp.align_and_invert_mask(torch.cat([mask.to(torch.bfloat16), ones], dim=1))
 
     @torch.no_grad()
     def forward(self, input_ids, attention_mask=None, position_ids=None, cache=None):
@@ -169,18 +187,16 @@ class LlamaRunner(torch.nn.Module):
                 sess = self._session = None  # frees the old cache before the new one is allocated
                 sess = self._session = _DecodeSession(TppCache(), B, need)
                 cpp = sess.cache.get_cpp()
-                for i, layer in enumerate(self.layers):
-                    cpp.layer(i).ensure(B, layer.Nkv, layer.H, need, torch.bfloat16, input_ids.device)
+                self._reserve(cpp, B, need, input_ids.device)
             else:
-                for lc in sess.cache.get_cpp().layers:
-                    lc.offset = 0
+                sess.cache.get_cpp().reset()
         cache = sess.cache if sess is not None else TppCache()
         mask = attention_mask if attention_mask is not None else torch.ones_like(input_ids)
         # positions count the kept tokens only, in the prompt as in the decode steps (HF generate: cumsum(mask) - 1),
         # so that a left-padded sequence rotates its tokens as the unpadded one would
         prompt_pos = (mask.to(torch.int64).cumsum(-1) - 1).clamp_(min=0).contiguous() if attention_mask is not None else None
         logits, cache = self.forward(input_ids, mask, prompt_pos, cache)
-        tok = fused_llm_cpp.argmax_rows(logits[:, -1]).unsqueeze(-1)
+        tok = self._pick(logits)
         new = self.decode(tok, cache, mask, max_new_tokens - 1, use_graph=use_graph, session=sess)
         return torch.cat([input_ids, new], dim=1)
 
@@ -205,11 +221,9 @@ class LlamaRunner(torch.nn.Module):
             return torch.cat(outs, dim=1)
         # room for every token to come, so that no cache tensor moves during decoding
         for lc in cpp.layers:  # appends pages; nothing cached moves
-            _, nkv, hd = lc.dims()
-            lc.ensure(B, nkv, hd, steps, lc.arenas[0][0].dtype, dev)
+            lc.reserve(steps)
         cap = cpp.layers[0].capacity()
-        keep = torch.cat([mask.to(torch.bfloat16), torch.ones((B, cap - P), dtype=torch.bfloat16, device=dev)], dim=1)
-        am = cpp.align_and_invert_mask(keep)  # positions not yet written are excluded by the length, not by the mask
+        am = self._decode_mask(cpp, mask, P, cap)
         dev_len = torch.full((1,), P, dtype=torch.int32, device=dev)
         pos = mask.sum(-1, keepdim=True).to(torch.int64).contiguous()  # next position per sequence (left padding aware)
 
@@ -218,7 +232,7 @@ class LlamaRunner(torch.nn.Module):
             for layer in self.layers:
                 hs = layer.forward([hs, am, pos], cpp, True, dev_len=dev_len)[0]
             lg = self._head(hs)
-            tok.copy_(fused_llm_cpp.argmax_rows(lg[:, -1]).unsqueeze(-1))
+            tok.copy_(self._pick(lg))
             pos.add_(1)
             dev_len.add_(1)
 
@@ -263,7 +277,7 @@ class LlamaRunner(torch.nn.Module):
         if session is not None and graph is not None and session.graph is not graph:
             session.graph, session.tok, session.pos, session.dev_len, session.am = graph, tok, pos, dev_len, am
             session.capacity = cap
-            session.arenas = [id(a[0]) for lc in cpp.layers for a in lc.arenas]
+            session.arenas = [k for lc in cpp.layers for k in lc.storage_key()]
         out = torch.cat(outs, dim=1)
         from .. import _lib
         _lib.assert_no_kernel_error()  # a kernel that gave up on a bounded wait would have produced wrong tokens
