@@ -103,30 +103,46 @@ typedef struct {
 } TpxLatentAbsorb;
 int tpx_latent_absorb(const TpxLatentAbsorb* a, void* stream);
 
-/* Softmax attention in the latent space: ol[T][heads][krp] fp32 = sum_j p_j c_j over the keys j of the token's window
+/* Softmax attention in the latent space: ol[T][heads][krp] = sum_j p_j c_j over the keys j of the token's window
  * (window tokens including itself), from the pages (lat == NULL, S == 1) or from lat [B][L][R]. */
 typedef struct {
   const void *qa, *lat;
   const uint64_t* pages;
   const int32_t *start, *dev_len;
-  float* ol;
+  void* ol;
   int64_t B, S, L, past, npages, heads, krp, R, window;
   float scale;
   int f32;
-  void* scratch; /* decode: zero before first use, left zero */
-  size_t scratch_bytes;
 } TpxLatentAttn;
 int tpx_latent_attn(const TpxLatentAttn* a, void* stream);
 
 /* out[T][ldo] = gate * (W_uv(head) ol), head by head; w_uv [heads * vdim][krp]; columns beyond heads * vdim set to zero. */
 typedef struct {
-  const float *ol, *gate;
+  const void* ol;
+  const float* gate;
   const void* w_uv;
   void* out;
   int64_t T, heads, vdim, krp, ldo;
   int f32;
 } TpxLatentValue;
 int tpx_latent_value(const TpxLatentValue* a, void* stream);
+
+/* Several bf16 tokens at once with keys and values expanded from the latents: out[T][ldo] = gate * softmax attention, window
+ * and keys as in tpx_latent_attn. kv [B * L][ldkv] holds, per row of lat, heads * dim keys and then heads * vdim values; q
+ * [T][ldq] is rotated in place. Runs on tcgen05; tpx_latent_prefill_serves says for which head sizes. The waits inside are
+ * bounded: tpx_latent_tc_status reads (and clears) the code of one that gave up. */
+typedef struct {
+  void* q;
+  const void *kv, *lat;
+  const float *cos_sin, *gate;
+  const int32_t* start;
+  void* out;
+  int64_t B, S, L, past, heads, dim, rot_dim, vdim, krp, R, ldq, ldkv, ldo, window;
+  float scale;
+} TpxLatentPrefill;
+int tpx_latent_prefill_serves(int64_t dim, int64_t rot_dim, int64_t vdim);
+int tpx_latent_prefill(const TpxLatentPrefill* a, void* stream);
+int tpx_latent_tc_status(void* stream, unsigned* status_host);
 
 /* Generalized delta rule over S tokens: per head and token, with u = k / sqrt(sum k^2 + 1e-6), decay w = exp(-e^(-1/2)
  * sigmoid(wraw)), rate a = sigmoid(araw + a_bias):  S <- diag(w) S - (a u)(u^T S) + k v^T,  o = S^T r; then o over its root

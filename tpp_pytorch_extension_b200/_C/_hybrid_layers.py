@@ -119,8 +119,8 @@ class LatentAttention:
 
     def __init__(self, w, heads, dim, rot_dim, vdim, kv_rank, window, scale, rot_base, eps, dtype, device, source=None, cache_window=None):
         self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = heads, dim, rot_dim, vdim, kv_rank
-        self.window, self.scale, self.eps, self.source, self.dtype = int(window), float(scale), float(eps), source, dtype
-        self.cache_window = int(cache_window or window)
+        self.window, self.scale, self.eps, self.source, self.dtype = min(int(window), 1 << 29), float(scale), float(eps), source, dtype
+        self.cache_window = min(int(cache_window or window), 1 << 29)
         mat = lambda t: t.to(device, dtype)
         vec = lambda t: t.to(device, torch.float32).contiguous()
         self.q_rank = w["dq"].shape[0]
@@ -133,6 +133,11 @@ class LatentAttention:
         self.uq = pad_matrix(mat(w["uq"]))
         self.uk = pad_matrix(mat(w["uk"]), 1, 16)
         self.uv = pad_matrix(mat(w["uv"]), 1, 16)
+        # keys and values of a multi-token call as one linear of the latents, where its kernel serves the head sizes
+        self.kv = None
+        if dtype == torch.bfloat16 and _lib.lib().tpx_latent_prefill_serves(dim, rot_dim, vdim):
+            self.kv = pad_matrix(torch.cat([self.uk, self.uv], 0))
+            self.uk, self.uv = self.kv[:heads * dim], self.kv[heads * dim:heads * (dim + vdim)]
         self.o = pad_matrix(mat(w["o"]), 1, 8)
         half = torch.arange(rot_dim // 2, dtype=torch.float64)
         self.freq = (float(rot_base) ** (-2.0 * half / max(rot_dim, 1))).to(device)
@@ -169,15 +174,22 @@ class LatentAttention:
             pages=src.ptrs.data_ptr(), B=B, S=S, L=L, ldp=proj.shape[1], ldq=cq.shape[1], past=past, npages=src.pages(), q_rank=self.q_rank,
             kv_rank=self.kv_rank, krp=self.krp, rot_dim=self.rot_dim, R=self.R, heads=self.heads, eps=self.eps, own_kv=int(self.source is None), f32=f32))
         q = linear(cq, self.uq)
+        out = torch.empty((T, self.o.shape[1]), dtype=self.dtype, device=dev)
+        if S > 1 and self.kv is not None:
+            kv = linear(lat.view(B * L, self.R)[:, :self.krp], self.kv)
+            _call("tpx_latent_prefill", _lib.LatentPrefillStruct(
+                q=q.data_ptr(), kv=kv.data_ptr(), lat=lat.data_ptr(), cos_sin=cos_sin.data_ptr(), gate=gate.data_ptr(), start=_lib.ptr(step.start),
+                out=out.data_ptr(), B=B, S=S, L=L, past=past, heads=self.heads, dim=self.dim, rot_dim=self.rot_dim, vdim=self.vdim, krp=self.krp, R=self.R,
+                ldq=q.shape[1], ldkv=kv.shape[1], ldo=out.shape[1], window=self.window, scale=self.scale))
+            return linear(out, self.o, out_f32=True)
         qa = torch.empty((T, self.heads, self.R), dtype=self.dtype, device=dev)
         _call("tpx_latent_absorb", _lib.LatentAbsorbStruct(
             q=q.data_ptr(), w_uk=self.uk.data_ptr(), cos_sin=cos_sin.data_ptr(), qa=qa.data_ptr(), T=T, ldq=q.shape[1], heads=self.heads, dim=self.dim,
             kv_rank=self.kv_rank, krp=self.krp, rot_dim=self.rot_dim, R=self.R, f32=f32))
-        ol = torch.empty((T, self.heads, self.krp), dtype=torch.float32, device=dev)
+        ol = torch.empty((T, self.heads, self.krp), dtype=self.dtype, device=dev)
         _call("tpx_latent_attn", _lib.LatentAttnStruct(
             qa=qa.data_ptr(), lat=_lib.ptr(lat), pages=src.ptrs.data_ptr(), start=_lib.ptr(step.start), dev_len=_lib.ptr(step.dev_len), ol=ol.data_ptr(),
             B=B, S=S, L=L, past=past, npages=src.pages(), heads=self.heads, krp=self.krp, R=self.R, window=self.window, scale=self.scale, f32=f32))
-        out = torch.empty((T, self.o.shape[1]), dtype=self.dtype, device=dev)
         _call("tpx_latent_value", _lib.LatentValueStruct(
             ol=ol.data_ptr(), gate=gate.data_ptr(), w_uv=self.uv.data_ptr(), out=out.data_ptr(), T=T, heads=self.heads, vdim=self.vdim, krp=self.krp,
             ldo=out.shape[1], f32=f32))

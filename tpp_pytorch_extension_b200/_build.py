@@ -23,7 +23,7 @@ NVCC_FLAGS = [
 
 
 # sources of models that do not need the whole library (names without the tpx_ prefix)
-COMPONENTS = {"Dofivik": ("api", "linear_bf16", "linear_f32", "postnorm", "latent", "delta")}
+COMPONENTS = {"Dofivik": ("api", "linear_bf16", "linear_f32", "postnorm", "latent", "latent_tc", "latent_dec", "delta")}
 
 
 def sources():

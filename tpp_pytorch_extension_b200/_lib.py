@@ -77,6 +77,9 @@ _SIGS = {
     "tpx_latent_absorb": (c_int, [c_vp, c_vp]),
     "tpx_latent_attn": (c_int, [c_vp, c_vp]),
     "tpx_latent_value": (c_int, [c_vp, c_vp]),
+    "tpx_latent_prefill_serves": (c_int, [c_i64] * 3),
+    "tpx_latent_prefill": (c_int, [c_vp, c_vp]),
+    "tpx_latent_tc_status": (c_int, [c_vp, ctypes.POINTER(ctypes.c_uint)]),
     "tpx_delta_rule": (c_int, [c_vp, c_vp]),
     "tpx_qlinear": (c_int, [c_int, c_vp, c_vp, c_vp, c_vp, c_i64, c_vp, c_i64, c_i64, c_i64, c_vp, c_int, c_vp, c_vp,
                             c_f32, c_vp, c_vp, c_sz, c_vp]),
@@ -142,9 +145,10 @@ PostnormFinalStruct = _struct("PostnormFinalStruct", p="x y w w_final rows out",
 LatentPrepStruct = _struct("LatentPrepStruct", p="proj q_norm kv_norm freq start dev_len cq cos_sin gate lat pages",
                            l="B S L ldp ldq past npages q_rank kv_rank krp rot_dim R heads", f="eps", i="own_kv f32")
 LatentAbsorbStruct = _struct("LatentAbsorbStruct", p="q w_uk cos_sin qa", l="T ldq heads dim kv_rank krp rot_dim R", i="f32")
-LatentAttnStruct = _struct("LatentAttnStruct", p="qa lat pages start dev_len ol", l="B S L past npages heads krp R window", f="scale", i="f32",
-                           p2="scratch", z="scratch_bytes")
+LatentAttnStruct = _struct("LatentAttnStruct", p="qa lat pages start dev_len ol", l="B S L past npages heads krp R window", f="scale", i="f32")
 LatentValueStruct = _struct("LatentValueStruct", p="ol gate w_uv out", l="T heads vdim krp ldo", i="f32")
+LatentPrefillStruct = _struct("LatentPrefillStruct", p="q kv lat cos_sin gate start out",
+                              l="B S L past heads dim rot_dim vdim krp R ldq ldkv ldo window", f="scale")
 DeltaRuleStruct = _struct("DeltaRuleStruct", p="proj wraw a_bias norm_w start dev_len state raw out", l="B S past ldp ldo heads dim", f="eps", i="f32")
 
 
@@ -206,11 +210,12 @@ def assert_no_kernel_error(sync=True):
         code = inst.error_code()
         if code:
             raise TpxError(f"the peer-memory all-reduce gave up waiting for rank {code - 1}")
-    if _lib is not None and hasattr(_lib, "tpx_attention_tc_status") and torch.cuda.is_available():
-        st = ctypes.c_uint(0)
-        check(_lib.tpx_attention_tc_status(stream(), ctypes.byref(st)))
-        if st.value:
-            raise TpxError(f"the prefill attention kernel gave up on a bounded wait (code {st.value})")
+    for name in ("tpx_attention_tc_status", "tpx_latent_tc_status"):
+        if _lib is not None and hasattr(_lib, name) and torch.cuda.is_available():
+            st = ctypes.c_uint(0)
+            check(getattr(_lib, name)(stream(), ctypes.byref(st)))
+            if st.value:
+                raise TpxError(f"a prefill attention kernel gave up on a bounded wait ({name}: code {st.value})")
 
 
 _scratch = {}

@@ -36,6 +36,7 @@ static void read_knobs() {
   g_knobs.tc_p_uks = env("TPX_TC_P_UKS", 2);
   g_knobs.attn_splits = env("TPX_ATTN_SPLITS", 0);
   g_knobs.attn_tc = env("TPX_ATTN_TC", 1);
+  g_knobs.pdl = env("TPX_PDL", 1) != 0;
 #ifdef TPX_DEBUG
   g_knobs.dbg = env("TPX_TC_DBG", 0);
 #else

@@ -46,6 +46,14 @@ __device__ __forceinline__ float hy_act(float v, int act, float a0, float a1) {
   }
 }
 
+// bf16 decoding of latent attention (tpx_latent_dec.cu)
+bool latent_absorb_mma_serves(const TpxLatentAbsorb& a);
+int latent_absorb_mma(const TpxLatentAbsorb& a, cudaStream_t st);
+bool latent_value_mma_serves(const TpxLatentValue& a);
+int latent_value_mma(const TpxLatentValue& a, cudaStream_t st);
+bool latent_decode_serves(const TpxLatentAttn& a);
+int latent_decode(const TpxLatentAttn& a, cudaStream_t st);
+
 // the bf16 operands of tpx_linear on the tcgen05 kernel (tpx_linear_bf16.cu)
 int linear_tc_ex(const TpxLinear& a, cudaStream_t st);
 

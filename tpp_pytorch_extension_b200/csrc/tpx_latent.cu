@@ -165,11 +165,11 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(TpxLatentAttn p) {
     for (int i = 0; i < NR; i++) acc[i] = fmaf(acc[i], al, pr * k[i]);
   }
   const float inv = l > 0.0f ? 1.0f / l : 0.0f;
-  float* o = p.ol + item * p.krp;
+  T* o = reinterpret_cast<T*>(p.ol) + item * p.krp;
 #pragma unroll
   for (int i = 0; i < NR; i++) {
     const int e = i * 32 + lane;
-    if (e < p.krp) o[e] = acc[i] * inv;
+    if (e < p.krp) hy_st(o + e, acc[i] * inv);
   }
 }
 
@@ -185,7 +185,7 @@ __global__ void __launch_bounds__(256) latent_value_kernel(TpxLatentValue p) {
   const int krp = (int)p.krp;
   for (int i = threadIdx.x; i < kAbsTok * krp; i += 256) {
     const int j = i / krp;
-    lv_o[i] = j < n ? p.ol[((t0 + j) * p.heads + head) * krp + i % krp] : 0.0f;
+    lv_o[i] = j < n ? hy_ld(reinterpret_cast<const T*>(p.ol) + ((t0 + j) * p.heads + head) * krp + i % krp) : 0.0f;
   }
   __syncthreads();
   T* out = reinterpret_cast<T*>(p.out);
@@ -258,6 +258,7 @@ extern "C" int tpx_latent_absorb(const TpxLatentAbsorb* a, void* stream) {
   TPX_REQUIRE(a->dim <= 1024, TPX_ERR_UNSUPPORTED, "latent_absorb: heads of at most 1024 channels");
   if (a->T == 0) return TPX_OK;
   TPX_REQUIRE(a->q && a->w_uk && a->qa && (a->rot_dim == 0 || a->cos_sin), TPX_ERR_ARG, "latent_absorb: null pointer");
+  if (latent_absorb_mma_serves(*a)) return latent_absorb_mma(*a, (cudaStream_t)stream);
   const int64_t tz = (a->T + kAbsTok - 1) / kAbsTok;
   TPX_REQUIRE(tz <= 65535, TPX_ERR_UNSUPPORTED, "latent_absorb: too many tokens in one call");
   const dim3 grid((unsigned)a->heads, (unsigned)((a->krp + 127) / 128), (unsigned)tz);
@@ -277,6 +278,7 @@ extern "C" int tpx_latent_attn(const TpxLatentAttn* a, void* stream) {
   TPX_REQUIRE(a->lat ? a->L >= a->S + (a->window - 1 < a->past ? a->window - 1 : a->past)
                      : a->S == 1 && a->pages && a->npages > 0, TPX_ERR_ARG, "latent_attn: the keys of the window are not there");
   TPX_REQUIRE(!a->dev_len || a->S == 1, TPX_ERR_ARG, "latent_attn: dev_len is for single tokens");
+  if (latent_decode_serves(*a)) return latent_decode(*a, (cudaStream_t)stream);
   return a->f32 ? latent_attn_plain<float>(*a, (cudaStream_t)stream) : latent_attn_plain<__nv_bfloat16>(*a, (cudaStream_t)stream);
 }
 
@@ -285,6 +287,7 @@ extern "C" int tpx_latent_value(const TpxLatentValue* a, void* stream) {
   TPX_REQUIRE(a->T >= 0 && a->heads > 0 && a->vdim > 0 && a->krp > 0 && a->krp <= 1152 && a->ldo >= a->heads * a->vdim, TPX_ERR_ARG, "latent_value: bad shape");
   if (a->T == 0) return TPX_OK;
   TPX_REQUIRE(a->ol && a->gate && a->w_uv && a->out, TPX_ERR_ARG, "latent_value: null pointer");
+  if (latent_value_mma_serves(*a)) return latent_value_mma(*a, (cudaStream_t)stream);
   const int64_t tz = (a->T + kAbsTok - 1) / kAbsTok;
   TPX_REQUIRE(tz <= 65535, TPX_ERR_UNSUPPORTED, "latent_value: too many tokens in one call");
   const dim3 grid((unsigned)a->heads, (unsigned)((a->vdim + 31) / 32), (unsigned)tz);

@@ -1,0 +1,427 @@
+// Decoding with latent attention in bf16: the per-head maps (keys into the query, latents into values) as small grouped
+// matrix products, and attention of all heads over the cached latents, each read once.
+//
+// Attention: a thread-block cluster per (sequence, group of 32 heads); its CTAs share the window's keys in tiles of 64.
+// A tile (64 latent rows of R values, through the page table) is staged by cp.async two deep. Eight warps: each computes
+// the scores of 8 keys for all heads, then the softmax of 4 heads, then the weighted sum of its eighth of the latent
+// columns for all heads (mma.sync bf16, fp32 accumulation; a latent row is key and value at once). The weights are
+// multiplied as two bf16 terms, so that they keep their 32-bit value in effect. The CTAs of a cluster merge through
+// distributed shared memory: nothing partial goes to global memory.
+#include "tpx_hybrid.cuh"
+#include "tpx_tc_ptx.cuh"
+
+namespace tpx {
+
+__device__ __forceinline__ void ld_cp16(uint32_t dst, const void* src, bool ok) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void ld_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void ld_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void ldm_x4(uint32_t a, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void ldm_x4t(uint32_t a, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void ldm_x2(uint32_t a, uint32_t (&r)[2]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void ldm_x2t(uint32_t a, uint32_t (&r)[2]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t ld_pack(float lo, float hi) {
+  __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+  return *reinterpret_cast<uint32_t*>(&v);
+}
+
+// ---------------------------------------------------------------- grouped products
+struct GroupedParams {
+  const uint16_t *w, *x;
+  uint16_t* out;
+  const float* gate;                // value map: [T][groups]
+  long long ldx, xg, ldo, og, ldw;  // strides: x token, x group, out token, out group, w row
+  int T, N, K, KP;                  // KP: K rounded up to 16
+  int groups;
+  // key map: the rotated query part
+  const float* cos_sin;
+  int dim, rot, krp, R;
+  long long pad0, pad1;             // value map: columns [pad0, pad1) of an output row are set to zero
+};
+
+// TRANS: w[group][k][n] (rows of one k), else w[group][n][k]. 4 warps x NT8 tiles of 8 outputs; 16 tokens at a time.
+template <int NT8, bool TRANS>
+__global__ void __launch_bounds__(128) grouped_mma_kernel(GroupedParams p) {
+  constexpr int NT = 32 * NT8;
+  extern __shared__ __align__(16) unsigned char gr_smem[];
+  const int g = blockIdx.x, n0 = blockIdx.y * NT;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int ldws = TRANS ? NT + 8 : p.KP + 8, ldxs = p.KP + 8;
+  uint16_t* sw = reinterpret_cast<uint16_t*>(gr_smem);
+  uint16_t* sx = sw + (size_t)(TRANS ? p.KP : NT) * ldws;
+  pdl_trigger();
+  if (TRANS && n0 >= p.N) {  // the last block of a group: the rotated part of the queries
+    pdl_wait();
+    const int rw = p.R - p.krp, half = p.rot / 2;
+    for (int i = threadIdx.x; i < p.T * rw; i += 128) {
+      const int j = i / rw, e = i % rw;
+      float v = 0.0f;
+      if (e < p.rot) {
+        const float2 r = reinterpret_cast<const float2*>(p.cos_sin)[(int64_t)j * half + (e >> 1)];
+        const uint16_t* qr = p.x + j * p.ldx + g * p.xg + p.dim;
+        const float a = bf16_bits_to_f32(qr[e & ~1]), b = bf16_bits_to_f32(qr[e | 1]);
+        v = (e & 1) ? b * r.x + a * r.y : a * r.x - b * r.y;
+      }
+      p.out[j * p.ldo + g * p.og + p.krp + e] = f32_to_bf16_bits(v);
+    }
+    return;
+  }
+  // weights do not depend on earlier kernels
+  if (TRANS) {
+    for (int i = threadIdx.x; i < p.KP * (NT / 8); i += 128) {
+      const int r = i / (NT / 8), c = (i % (NT / 8)) * 8;
+      const bool ok = r < p.K && n0 + c < p.N;
+      ld_cp16(tc_smem_u32(sw + r * ldws + c), ok ? p.w + ((long long)g * p.K + r) * p.ldw + n0 + c : p.w, ok);
+    }
+  } else {
+    const int kc = p.KP / 8;
+    for (int i = threadIdx.x; i < NT * kc; i += 128) {
+      const int r = i / kc, c = (i % kc) * 8;
+      const bool ok = n0 + r < p.N;
+      ld_cp16(tc_smem_u32(sw + r * ldws + c), ok ? p.w + ((long long)g * p.N + n0 + r) * p.ldw + c : p.w, ok);
+    }
+  }
+  ld_commit();
+  pdl_wait();
+  const int kc = p.KP / 8;
+  for (int t0 = 0; t0 < p.T; t0 += 16) {
+    if (t0) __syncthreads();
+    for (int i = threadIdx.x; i < 16 * kc; i += 128) {
+      const int r = i / kc, c = (i % kc) * 8;
+      const bool ok = t0 + r < p.T && c < p.K;
+      ld_cp16(tc_smem_u32(sx + r * ldxs + c), ok ? p.x + (t0 + r) * p.ldx + g * p.xg + c : p.x, ok);
+    }
+    ld_commit();
+    ld_wait<0>();
+    __syncthreads();
+    float acc[NT8][4] = {};
+    const uint32_t xa = tc_smem_u32(sx + (lane & 15) * ldxs + (lane >> 4) * 8);
+    for (int k = 0; k < p.KP; k += 16) {
+      uint32_t a[4];
+      ldm_x4(xa + k * 2, a);
+#pragma unroll
+      for (int i = 0; i < NT8; i++) {
+        const int n = (warp * NT8 + i) * 8;
+        uint32_t b[2];
+        if (TRANS) ldm_x2t(tc_smem_u32(sw + (k + (lane & 15)) * ldws + n), b);
+        else ldm_x2(tc_smem_u32(sw + (n + (lane & 7)) * ldws + k + ((lane >> 3) & 1) * 8), b);
+        mma16816(acc[i], a, b[0], b[1]);
+      }
+    }
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+      const int t = t0 + (lane >> 2) + h * 8;
+      if (t < p.T) {
+        const float s = p.gate ? p.gate[(long long)t * p.groups + g] : 1.0f;
+#pragma unroll
+        for (int i = 0; i < NT8; i++) {
+          const int n = n0 + (warp * NT8 + i) * 8 + (lane & 3) * 2;
+          uint16_t* o = p.out + t * p.ldo + g * p.og + n;
+          if (n < p.N) o[0] = f32_to_bf16_bits(acc[i][2 * h] * s);
+          if (n + 1 < p.N) o[1] = f32_to_bf16_bits(acc[i][2 * h + 1] * s);
+        }
+      }
+    }
+  }
+  if (!TRANS && g == 0 && blockIdx.y == 0)
+    for (int t = 0; t < p.T; t++)
+      for (long long c = p.pad0 + threadIdx.x; c < p.pad1; c += 128) p.out[t * p.ldo + c] = 0;
+}
+
+template <int NT8, bool TRANS>
+static int grouped_launch(const GroupedParams& p, int extra_blocks, cudaStream_t st) {
+  constexpr int NT = 32 * NT8;
+  const size_t smem = ((size_t)(TRANS ? p.KP : NT) * (TRANS ? NT + 8 : p.KP + 8) + (size_t)16 * (p.KP + 8)) * 2;
+  TPX_REQUIRE(smem <= 220 * 1024, TPX_ERR_UNSUPPORTED, "latent decode: per-head map too large (contraction of %d)", p.K);
+  static bool opted[16] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 16 || !opted[dev]) {
+    TPX_CUDA_OK(cudaFuncSetAttribute(grouped_mma_kernel<NT8, TRANS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    if (dev >= 0 && dev < 16) opted[dev] = true;
+  }
+  TPX_CUDA_OK(launch_pdl(grouped_mma_kernel<NT8, TRANS>, dim3((unsigned)p.groups, (unsigned)((p.N + NT - 1) / NT + extra_blocks)), dim3(128), smem, st, p));
+  return TPX_OK;
+}
+
+bool latent_absorb_mma_serves(const TpxLatentAbsorb& a) {
+  return !a.f32 && a.T <= 64 && a.dim % 8 == 0 && (a.dim + a.rot_dim) % 8 == 0 && a.ldq % 8 == 0 && a.krp % 8 == 0 && a.dim <= 512 &&
+         (((uintptr_t)a.q | (uintptr_t)a.w_uk) & 15) == 0;
+}
+int latent_absorb_mma(const TpxLatentAbsorb& a, cudaStream_t st) {
+  GroupedParams p = {};
+  p.w = (const uint16_t*)a.w_uk; p.x = (const uint16_t*)a.q; p.out = (uint16_t*)a.qa;
+  p.ldx = a.ldq; p.xg = a.dim + a.rot_dim; p.ldo = a.heads * a.R; p.og = a.R; p.ldw = a.krp;
+  p.T = (int)a.T; p.N = (int)a.krp; p.K = (int)a.dim; p.KP = (int)((a.dim + 15) / 16 * 16); p.groups = (int)a.heads;
+  p.cos_sin = a.cos_sin; p.dim = (int)a.dim; p.rot = (int)a.rot_dim; p.krp = (int)a.krp; p.R = (int)a.R;
+  return grouped_launch<2, true>(p, a.R > a.krp ? 1 : 0, st);
+}
+bool latent_value_mma_serves(const TpxLatentValue& a) {
+  return !a.f32 && a.T <= 64 && a.krp % 16 == 0 && a.krp <= 1152 && (((uintptr_t)a.ol | (uintptr_t)a.w_uv) & 15) == 0;
+}
+int latent_value_mma(const TpxLatentValue& a, cudaStream_t st) {
+  GroupedParams p = {};
+  p.w = (const uint16_t*)a.w_uv; p.x = (const uint16_t*)a.ol; p.out = (uint16_t*)a.out; p.gate = a.gate;
+  p.ldx = a.heads * a.krp; p.xg = a.krp; p.ldo = a.ldo; p.og = a.vdim; p.ldw = a.krp;
+  p.T = (int)a.T; p.N = (int)a.vdim; p.K = (int)a.krp; p.KP = (int)a.krp; p.groups = (int)a.heads;
+  p.pad0 = a.heads * a.vdim; p.pad1 = a.ldo;
+  return grouped_launch<1, false>(p, 0, st);
+}
+
+// ---------------------------------------------------------------- attention
+constexpr int kLdKeys = 64, kLdWarps = 8, kLdThreads = 256;
+
+// MT: 16-head tiles per CTA. CW: latent columns per warp / 8 (fits krp <= CW * 64)
+template <int MT, int CW>
+__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentAttn p, int splits) {
+  constexpr int MR = MT * 16;
+  extern __shared__ __align__(16) unsigned char ld_smem[];
+  const int R = (int)p.R, krp = (int)p.krp, lds = R + 8;
+  uint16_t* sk = reinterpret_cast<uint16_t*>(ld_smem);                 // [2][64][R + 8]
+  uint16_t* sq = sk + (size_t)2 * kLdKeys * lds;                       // [MR][R + 8]
+  uint16_t* sp = sq + (size_t)MR * lds;                                // [2 terms][MR][64 + 8]
+  float* ss = reinterpret_cast<float*>(sp + 2 * MR * (kLdKeys + 8));   // [MR][64 + 4]
+  float* sm = ss + MR * (kLdKeys + 4);                                 // [MR] running maxima (log2 units)
+  float* sl = sm + MR;                                                 // [MR] running sums
+  float* sa = sl + MR;                                                 // [MR] rescaling of this tile
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int rank = blockIdx.x % splits, b = blockIdx.x / splits, h0 = blockIdx.y * MR;
+  pdl_trigger();
+  pdl_wait();
+  const int64_t t = p.dev_len ? *p.dev_len : p.past;
+  const int64_t lo = max((int64_t)(p.start ? p.start[b] : 0), t - p.window + 1);
+  const int tiles = (int)((t - lo + kLdKeys) / kLdKeys);  // ceil((t - lo + 1) / 64)
+  const int i0 = (int)((long long)tiles * rank / splits), i1 = (int)((long long)tiles * (rank + 1) / splits);
+
+  const int rc = R / 8;
+  for (int i = threadIdx.x; i < MR * rc; i += kLdThreads) {
+    const int r = i / rc, c = (i % rc) * 8;
+    const bool ok = h0 + r < p.heads;
+    const uint16_t* q = reinterpret_cast<const uint16_t*>(p.qa);
+    ld_cp16(tc_smem_u32(sq + r * lds + c), ok ? q + ((int64_t)b * p.heads + h0 + r) * R + c : q, ok);
+  }
+  auto fetch = [&](int i, int stage) {  // a warp per key row
+#pragma unroll
+    for (int rr = 0; rr < kLdKeys / kLdWarps; rr++) {
+      const int r = warp * (kLdKeys / kLdWarps) + rr;
+      const int64_t j = lo + (int64_t)i * kLdKeys + r;
+      const bool ok = j <= t;
+      const int64_t jj = ok ? j : t;
+      const uint16_t* src = reinterpret_cast<const uint16_t*>(__ldg(p.pages + (jj / 32) % p.npages)) + ((int64_t)b * 32 + jj % 32) * R;
+      for (int c = lane; c < rc; c += 32) ld_cp16(tc_smem_u32(sk + ((size_t)stage * kLdKeys + r) * lds + c * 8), src + c * 8, ok);
+    }
+    ld_commit();
+  };
+  for (int i = threadIdx.x; i < MR; i += kLdThreads) { sm[i] = -INFINITY; sl[i] = 0.0f; }
+  float o[MT][CW][4];
+#pragma unroll
+  for (int m = 0; m < MT; m++)
+#pragma unroll
+    for (int c = 0; c < CW; c++)
+#pragma unroll
+      for (int e = 0; e < 4; e++) o[m][c][e] = 0.0f;
+  const float sc2 = p.scale * 1.4426950408889634f;
+  const int cols = (krp / 8 + kLdWarps - 1) / kLdWarps;  // 8-column tiles per warp
+  const int ct0 = warp * cols;
+  if (i0 < i1) fetch(i0, 0);
+  else ld_commit();
+  for (int i = i0; i < i1; i++) {
+    const int stage = (i - i0) & 1;
+    ld_wait<0>();
+    __syncthreads();  // tile i is there, and nobody still reads the other stage or the weights of tile i - 1
+    if (i + 1 < i1) fetch(i + 1, stage ^ 1);
+    const uint16_t* kt = sk + (size_t)stage * kLdKeys * lds;
+    {  // scores of this warp's 8 keys
+      float acc[MT][4] = {};
+      const uint32_t kb = tc_smem_u32(kt + (warp * 8 + (lane & 7)) * lds + ((lane >> 3) & 1) * 8);
+      const uint32_t qa = tc_smem_u32(sq + (lane & 15) * lds + (lane >> 4) * 8);
+#pragma unroll 4
+      for (int k = 0; k < R; k += 16) {
+        uint32_t bb[2];
+        ldm_x2(kb + k * 2, bb);
+#pragma unroll
+        for (int m = 0; m < MT; m++) {
+          uint32_t a[4];
+          ldm_x4(qa + (m * 16 * lds + k) * 2, a);
+          mma16816(acc[m], a, bb[0], bb[1]);
+        }
+      }
+      const int key = warp * 8 + (lane & 3) * 2;
+      const int64_t left = t - (lo + (int64_t)i * kLdKeys);  // keys 0 .. left exist
+#pragma unroll
+      for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+          float* d = ss + (m * 16 + (lane >> 2) + h * 8) * (kLdKeys + 4) + key;
+          d[0] = key <= left ? acc[m][2 * h] * sc2 : -INFINITY;
+          d[1] = key + 1 <= left ? acc[m][2 * h + 1] * sc2 : -INFINITY;
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int rr = 0; rr < MR / kLdWarps; rr++) {  // softmax of this warp's heads, two keys per lane
+      const int r = warp * (MR / kLdWarps) + rr;
+      const float x0 = ss[r * (kLdKeys + 4) + lane * 2], x1 = ss[r * (kLdKeys + 4) + lane * 2 + 1];
+      float mx = fmaxf(x0, x1);
+#pragma unroll
+      for (int s = 16; s > 0; s >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, s));
+      const float mo = sm[r], mn = fmaxf(mo, mx);  // a tile has at least one key
+      const float e0 = exp2f(x0 - mn), e1 = exp2f(x1 - mn), al = exp2f(mo - mn);
+      const float sum = hy_warp_sum(e0 + e1);
+      const uint32_t hi = ld_pack(e0, e1);
+      const uint32_t low = ld_pack(e0 - __uint_as_float(hi << 16), e1 - __uint_as_float(hi & 0xffff0000u));
+      *reinterpret_cast<uint32_t*>(sp + r * (kLdKeys + 8) + lane * 2) = hi;
+      *reinterpret_cast<uint32_t*>(sp + (MR + r) * (kLdKeys + 8) + lane * 2) = low;
+      __syncwarp();
+      if (lane == 0) { sm[r] = mn; sl[r] = sl[r] * al + sum; sa[r] = al; }
+    }
+    __syncthreads();
+    // weighted sum of this warp's latent columns
+#pragma unroll
+    for (int m = 0; m < MT; m++) {
+      const float a0 = sa[m * 16 + (lane >> 2)], a1 = sa[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+      for (int c = 0; c < CW; c++) { o[m][c][0] *= a0; o[m][c][1] *= a0; o[m][c][2] *= a1; o[m][c][3] *= a1; }
+    }
+#pragma unroll
+    for (int k = 0; k < kLdKeys; k += 16) {
+      uint32_t a[MT][2][4];
+#pragma unroll
+      for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int term = 0; term < 2; term++)
+          ldm_x4(tc_smem_u32(sp + (term * MR + m * 16 + (lane & 15)) * (kLdKeys + 8) + k + (lane >> 4) * 8), a[m][term]);
+#pragma unroll
+      for (int c = 0; c < CW; c++) {
+        if (c < cols && (ct0 + c) * 8 < krp) {
+          uint32_t bb[2];
+          ldm_x2t(tc_smem_u32(kt + (k + (lane & 15)) * lds + (ct0 + c) * 8), bb);
+#pragma unroll
+          for (int m = 0; m < MT; m++) {
+            mma16816(o[m][c], a[m][0], bb[0], bb[1]);
+            mma16816(o[m][c], a[m][1], bb[0], bb[1]);
+          }
+        }
+      }
+    }
+  }
+  // merge: every CTA scales its sums to the cluster's maximum and total, then adds up its share of the columns
+  ld_wait<0>();
+  __syncthreads();
+  tc_cluster_sync();
+  float* so = reinterpret_cast<float*>(ld_smem);  // [MR][krp], over the key stages
+  for (int r = threadIdx.x; r < MR; r += kLdThreads) {
+    float mx = -INFINITY;
+    for (int c = 0; c < splits; c++) {
+      float v;
+      asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(tc_mapa(tc_smem_u32(sm + r), c)) : "memory");
+      mx = fmaxf(mx, v);
+    }
+    float tot = 0.0f;
+    for (int c = 0; c < splits; c++) {
+      float v, l;
+      asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(tc_mapa(tc_smem_u32(sm + r), c)) : "memory");
+      asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(l) : "r"(tc_mapa(tc_smem_u32(sl + r), c)) : "memory");
+      if (l > 0.0f) tot += l * exp2f(v - mx);
+    }
+    sa[r] = sl[r] > 0.0f ? exp2f(sm[r] - mx) / tot : 0.0f;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int m = 0; m < MT; m++) {
+    const int r = m * 16 + (lane >> 2);
+    const float a0 = sa[r], a1 = sa[r + 8];
+#pragma unroll
+    for (int c = 0; c < CW; c++) {
+      const int n = (ct0 + c) * 8 + (lane & 3) * 2;
+      if (c < cols && n < krp) {
+        so[r * krp + n] = o[m][c][0] * a0;
+        so[r * krp + n + 1] = o[m][c][1] * a0;
+        so[(r + 8) * krp + n] = o[m][c][2] * a1;
+        so[(r + 8) * krp + n + 1] = o[m][c][3] * a1;
+      }
+    }
+  }
+  tc_cluster_sync();
+  const int nq = MR * krp / 4;
+  for (int q = rank * kLdThreads + threadIdx.x; q < nq; q += splits * kLdThreads) {
+    float4 s = make_float4(0, 0, 0, 0);
+    for (int c = 0; c < splits; c++) {
+      const float4 v = tc_ld_cluster_f4(tc_mapa(tc_smem_u32(so + q * 4), c));
+      s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
+    }
+    const int r = q * 4 / krp, n = q * 4 % krp;
+    if (h0 + r < p.heads)
+      *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(p.ol) + ((int64_t)b * p.heads + h0 + r) * krp + n) = make_uint2(ld_pack(s.x, s.y), ld_pack(s.z, s.w));
+  }
+  tc_cluster_sync();  // nobody leaves while its shared memory is being read
+}
+
+static size_t ld_smem_bytes(int MR, int R) {
+  return ((size_t)2 * kLdKeys * (R + 8) + (size_t)MR * (R + 8) + 2 * MR * (kLdKeys + 8)) * 2 + (size_t)MR * (kLdKeys + 4) * 4 + 3 * MR * 4;
+}
+
+bool latent_decode_serves(const TpxLatentAttn& a) {
+  if (a.f32 || a.lat || a.S != 1 || a.R % 16 || a.krp % 16 || a.krp > 512) return false;
+  const int MR = a.heads <= 16 ? 16 : 32;
+  const size_t smem = ld_smem_bytes(MR, (int)a.R);
+  return smem <= 225 * 1024 && (size_t)MR * a.krp * 4 <= (size_t)2 * kLdKeys * (a.R + 8) * 2 && (((uintptr_t)a.qa | (uintptr_t)a.ol) & 15) == 0;
+}
+
+template <int MT, int CW>
+static int latent_decode_launch(const TpxLatentAttn& a, int splits, cudaStream_t st) {
+  const size_t smem = ld_smem_bytes(MT * 16, (int)a.R);
+  static bool opted[16] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 16 || !opted[dev]) {
+    TPX_CUDA_OK(cudaFuncSetAttribute(latent_decode_kernel<MT, CW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024));
+    if (dev >= 0 && dev < 16) opted[dev] = true;
+  }
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3((unsigned)(a.B * splits), (unsigned)((a.heads + MT * 16 - 1) / (MT * 16)));
+  cfg.blockDim = dim3(kLdThreads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = knobs().pdl;
+  attr[1].id = cudaLaunchAttributeClusterDimension;
+  attr[1].val.clusterDim.x = (unsigned)splits;
+  attr[1].val.clusterDim.y = 1;
+  attr[1].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 2;
+  count_launch();
+  TPX_CUDA_OK(cudaLaunchKernelEx(&cfg, latent_decode_kernel<MT, CW>, a, splits));
+  return TPX_OK;
+}
+
+int latent_decode(const TpxLatentAttn& a, cudaStream_t st) {
+  // keys that may be in the window (planning only; the kernel reads the count itself)
+  int64_t keys = a.npages * 32 < a.window ? a.npages * 32 : a.window;
+  if (!a.dev_len && a.past + 1 < keys) keys = a.past + 1;
+  const int64_t tiles = (keys + kLdKeys - 1) / kLdKeys, groups = (a.heads + 31) / 32;
+  int splits = 1;
+  while (splits < 8 && splits * 2 <= tiles && a.B * groups * splits * 2 <= sm_count() + sm_count() / 8) splits *= 2;
+  const int cw = (int)((a.krp / 8 + kLdWarps - 1) / kLdWarps);
+  if (a.heads <= 16) return cw <= 2 ? latent_decode_launch<1, 2>(a, splits, st) : cw <= 4 ? latent_decode_launch<1, 4>(a, splits, st) : latent_decode_launch<1, 8>(a, splits, st);
+  return cw <= 2 ? latent_decode_launch<2, 2>(a, splits, st) : cw <= 4 ? latent_decode_launch<2, 4>(a, splits, st) : latent_decode_launch<2, 8>(a, splits, st);
+}
+
+}  // namespace tpx
