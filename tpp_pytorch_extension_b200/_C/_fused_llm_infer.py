@@ -86,6 +86,16 @@ def _int8_tc(x, y, w, w2, bias, act, mul_in, res, res_scale, norm=None):
     return y
 
 
+def bf16_linear_scratch(M):
+    """Scratch of the bf16 linear for M rows and any weight: one size for all shapes, so that the buffer does not grow
+    between the layers of a step."""
+    key = ("bf16", 64 if M <= 64 else 0)
+    nb = _SCRATCH_BYTES.get(key)
+    if nb is None:
+        nb = _SCRATCH_BYTES[key] = max(_lib.lib().tpx_linear_bf16_tc_scratch_bytes(key[1] or 65, n, 4096) for n in (128, 128 * 149))
+    return nb
+
+
 def _bf16_linear(x, w, bias, act, mul_in, res, res_scale):
     """Unquantized bf16 weight, plain [N, K] (nn.Linear.weight) or blocked 5-D [N/bk, K/bc, bc/2, bk, 2]
     (BlockedParameter.block(), un-blocked once and cached on the tensor): tpx_linear_bf16_tc."""
@@ -116,7 +126,7 @@ def _bf16_linear(x, w, bias, act, mul_in, res, res_scale):
             _lib.require_cuda(t, name)
             if t.dtype != torch.bfloat16:
                 raise _lib.TpxError(f"fc_plain: {name} must be bfloat16")
-    sc = _lib.scratch(1 << 16, x.device)
+    sc = _lib.scratch(bf16_linear_scratch(M), x.device)
     _lib.check(_lib.lib().tpx_linear_bf16_tc(w.data_ptr(), x.data_ptr(), M, N, K, _lib.ptr(bias), ACT[act], _lib.ptr(mul_in),
                                              _lib.ptr(res), float(res_scale), y.data_ptr(), sc.data_ptr(), sc.numel(), _lib.stream()))
     return y

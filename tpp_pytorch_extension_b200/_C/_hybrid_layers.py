@@ -10,6 +10,7 @@ import torch
 
 from .. import _lib
 from .. import _timers
+from ._fused_llm_infer import bf16_linear_scratch
 
 ACT = {None: 0, "gelu": 1, "silu": 2, "relu": 3, "tanh": 4, "xielu": 5}
 
@@ -42,7 +43,7 @@ def linear(x, w, bias=None, act=None, act_from=0, act_params=None, out_f32=False
     y = torch.empty((M, N), dtype=torch.float32 if (f32 or out_f32) else torch.bfloat16, device=x.device)
     if x.dtype != w.dtype or x.shape[1] != K:
         raise _lib.TpxError(f"linear: input {tuple(x.shape)} {x.dtype} does not fit the weight {tuple(w.shape)} {w.dtype}")
-    sc = _lib.scratch(1 << 16, x.device)
+    sc = _lib.scratch(bf16_linear_scratch(M), x.device)
     _call("tpx_linear", _lib.LinearStruct(
         w=w.data_ptr(), x=x.data_ptr(), bias=_lib.ptr(bias), act_params=_lib.ptr(act_params), y=y.data_ptr(), M=M, N=N, K=K,
         ldw=w.stride(0), ldx=x.stride(0), ldy=N, f32=int(f32), out_f32=int(y.dtype == torch.float32), act=ACT[act], act_from=act_from,

@@ -7,60 +7,68 @@
 namespace tpx {
 
 // ---------------------------------------------------------------- norms, rotation, cache append: a CTA per token
+constexpr int kPrepThreads = 256;
 template <typename T>
-__global__ void __launch_bounds__(128) latent_prep_kernel(TpxLatentPrep p) {
-  __shared__ float red[32];
+__global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(TpxLatentPrep p) {
+  __shared__ float red[2][kPrepThreads / 32];
   pdl_trigger();
   pdl_wait();
   const int64_t row = blockIdx.x;
   const int b = (int)(row / p.S), s = (int)(row % p.S);
-  const float* x = p.proj + row * p.ldp;
+  const int q_rank = (int)p.q_rank, kv_rank = (int)p.kv_rank, krp = (int)p.krp, rot = (int)p.rot_dim;
+  const float* __restrict__ x = p.proj + row * p.ldp;
+  const float* __restrict__ xk = x + q_rank;
   const int64_t past = p.dev_len ? *p.dev_len : p.past;
   const int64_t t = past + s;
   const int64_t pos = t - (p.start ? p.start[b] : 0);  // negative: padding
-  // query latent
-  float ss = 0.0f;
-  for (int i = threadIdx.x; i < p.q_rank; i += 128) ss = fmaf(x[i], x[i], ss);
-  float inv = 1.0f / sqrtf(hy_block_sum(ss, red) / (float)p.q_rank + p.eps);
-  T* cq = reinterpret_cast<T*>(p.cq) + row * p.ldq;
-  for (int i = threadIdx.x; i < p.ldq; i += 128) hy_st(cq + i, i < p.q_rank ? x[i] * inv * p.q_norm[i] : 0.0f);
-  x += p.q_rank;
   // angles: the product position * frequency and its reduction to one turn in double, the functions in 32-bit
-  const int half = (int)p.rot_dim / 2;
-  float2* cs = reinterpret_cast<float2*>(p.cos_sin) + row * half;
-  for (int i = threadIdx.x; i < half; i += 128) {
-    const double a = (double)(pos > 0 ? pos : 0) * p.freq[i];
-    const double turns = a * 0.15915494309189533577;
+  float2* cs = reinterpret_cast<float2*>(p.cos_sin) + row * (rot / 2);
+  for (int i = threadIdx.x; i < rot / 2; i += kPrepThreads) {
+    const double turns = (double)(pos > 0 ? pos : 0) * p.freq[i] * 0.15915494309189533577;
     float sn, c;
     sincospif((float)(2.0 * (turns - rint(turns))), &sn, &c);
     cs[i] = make_float2(c, sn);
   }
+  float sq = 0.0f, sk = 0.0f;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < q_rank; i += kPrepThreads) sq = fmaf(x[i], x[i], sq);
+  if (p.own_kv)
+    for (int i = threadIdx.x; i < kv_rank; i += kPrepThreads) sk = fmaf(xk[i], xk[i], sk);
+  sq = hy_warp_sum(sq);
+  sk = hy_warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sk; }
+  __syncthreads();  // also publishes cs within the block
+  sq = sk = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kPrepThreads / 32; i++) { sq += red[0][i]; sk += red[1][i]; }
+  const float qi = 1.0f / sqrtf(sq / (float)q_rank + p.eps);
+  T* cq = reinterpret_cast<T*>(p.cq) + row * p.ldq;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < p.ldq; i += kPrepThreads) hy_st(cq + i, i < q_rank ? x[i] * qi * p.q_norm[i] : 0.0f);
   if (p.own_kv) {
-    ss = 0.0f;
-    for (int i = threadIdx.x; i < p.kv_rank; i += 128) ss = fmaf(x[i], x[i], ss);
-    inv = 1.0f / sqrtf(hy_block_sum(ss, red) / (float)p.kv_rank + p.eps);  // its barriers also publish cs
+    const float ki = 1.0f / sqrtf(sk / (float)kv_rank + p.eps);
     T* lat = p.lat ? reinterpret_cast<T*>(p.lat) + ((int64_t)b * p.L + (p.L - p.S) + s) * p.R : nullptr;
     // of the call's tokens only the last npages blocks stay in the cache: the others would be overwritten
     const int64_t last_block = (past + p.S - 1) / 32;
     T* page = t / 32 > last_block - p.npages
                   ? reinterpret_cast<T*>(p.pages[(t / 32) % p.npages]) + ((int64_t)b * 32 + t % 32) * p.R : nullptr;
-    for (int i = threadIdx.x; i < p.R; i += 128) {
+    for (int i = threadIdx.x; i < p.R; i += kPrepThreads) {
       float v = 0.0f;
-      if (i < p.kv_rank) {
-        v = x[i] * inv * p.kv_norm[i];
-      } else if (i >= p.krp && i < p.krp + p.rot_dim) {
-        const int e = i - (int)p.krp;
+      if (i < kv_rank) {
+        v = xk[i] * ki * p.kv_norm[i];
+      } else if (i >= krp && i < krp + rot) {
+        const int e = i - krp;
         const float2 r = cs[e >> 1];
-        const float u = x[p.kv_rank + (e & ~1)], w = x[p.kv_rank + (e | 1)];
+        const float u = xk[kv_rank + (e & ~1)], w = xk[kv_rank + (e | 1)];
         v = (e & 1) ? w * r.x + u * r.y : u * r.x - w * r.y;
       }
       if (pos < 0) v = 0.0f;
       if (lat) hy_st(lat + i, v);
       if (page) hy_st(page + i, v);
     }
-    x += p.kv_rank + p.rot_dim;
+    xk += kv_rank + rot;
   }
-  for (int i = threadIdx.x; i < p.heads; i += 128) p.gate[row * p.heads + i] = hy_sigmoid(x[i]);
+  for (int i = threadIdx.x; i < p.heads; i += kPrepThreads) p.gate[row * p.heads + i] = hy_sigmoid(xk[i]);
 }
 
 template <typename T>
@@ -235,8 +243,8 @@ extern "C" int tpx_latent_prep(const TpxLatentPrep* a, void* stream) {
               "latent_prep: a row is smaller than its contents");
   TPX_REQUIRE(!a->dev_len || a->S == 1, TPX_ERR_ARG, "latent_prep: dev_len is for single tokens");
   const dim3 grid((unsigned)(a->B * a->S));
-  if (a->f32) TPX_CUDA_OK(launch_pdl(latent_prep_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, *a));
-  else TPX_CUDA_OK(launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, dim3(128), 0, (cudaStream_t)stream, *a));
+  if (a->f32) TPX_CUDA_OK(launch_pdl(latent_prep_kernel<float>, grid, dim3(kPrepThreads), 0, (cudaStream_t)stream, *a));
+  else TPX_CUDA_OK(launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, dim3(kPrepThreads), 0, (cudaStream_t)stream, *a));
   return TPX_OK;
 }
 

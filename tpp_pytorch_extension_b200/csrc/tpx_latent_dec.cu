@@ -3,8 +3,9 @@
 //
 // Attention: a thread-block cluster per (sequence, group of 32 heads); its CTAs share the window's keys in tiles of 64.
 // A tile (64 latent rows of R values, through the page table) is staged by cp.async two deep. Eight warps: each computes
-// the scores of 8 keys for all heads, then the softmax of 4 heads, then the weighted sum of its eighth of the latent
-// columns for all heads (mma.sync bf16, fp32 accumulation; a latent row is key and value at once). The weights are
+// the part of the scores of 32 keys and all heads that a quarter of the row contributes (its slice of the queries stays in
+// registers: read from shared memory by every warp it would be the largest traffic there), then the softmax of 4 heads, then
+// the weighted sum of its eighth of the latent columns for all heads (mma.sync bf16, fp32 accumulation; a latent row is key and value at once). The weights are
 // multiplied as two bf16 terms, so that they keep their 32-bit value in effect. The CTAs of a cluster merge through
 // distributed shared memory: nothing partial goes to global memory.
 #include "tpx_hybrid.cuh"
@@ -186,47 +187,55 @@ int latent_value_mma(const TpxLatentValue& a, cudaStream_t st) {
 // ---------------------------------------------------------------- attention
 constexpr int kLdKeys = 64, kLdWarps = 8, kLdThreads = 256;
 
-// MT: 16-head tiles per CTA. CW: latent columns per warp / 8 (fits krp <= CW * 64)
-template <int MT, int CW>
+// MT: 16-head tiles per CTA; CW: 8-column latent tiles per warp (krp <= CW * 64); KS: 16-value steps of a quarter row
+template <int MT, int CW, int KS>
 __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentAttn p, int splits) {
-  constexpr int MR = MT * 16;
+  constexpr int MR = MT * 16, SW = kLdKeys + 4;
   extern __shared__ __align__(16) unsigned char ld_smem[];
   const int R = (int)p.R, krp = (int)p.krp, lds = R + 8;
   uint16_t* sk = reinterpret_cast<uint16_t*>(ld_smem);                 // [2][64][R + 8]
-  uint16_t* sq = sk + (size_t)2 * kLdKeys * lds;                       // [MR][R + 8]
-  uint16_t* sp = sq + (size_t)MR * lds;                                // [2 terms][MR][64 + 8]
-  float* ss = reinterpret_cast<float*>(sp + 2 * MR * (kLdKeys + 8));   // [MR][64 + 4]
-  float* sm = ss + MR * (kLdKeys + 4);                                 // [MR] running maxima (log2 units)
+  uint16_t* sp = sk + (size_t)2 * kLdKeys * lds;                       // [2 terms][MR][64 + 8]
+  float* ss = reinterpret_cast<float*>(sp + 2 * MR * (kLdKeys + 8));   // [4 quarters][MR][64 + 4]
+  float* sm = ss + 4 * MR * SW;                                        // [MR] running maxima (log2 units)
   float* sl = sm + MR;                                                 // [MR] running sums
   float* sa = sl + MR;                                                 // [MR] rescaling of this tile
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int rank = blockIdx.x % splits, b = blockIdx.x / splits, h0 = blockIdx.y * MR;
+  const int kq = warp & 3, key0 = (warp >> 2) * 32;
   pdl_trigger();
   pdl_wait();
   const int64_t t = p.dev_len ? *p.dev_len : p.past;
   const int64_t lo = max((int64_t)(p.start ? p.start[b] : 0), t - p.window + 1);
   const int tiles = (int)((t - lo + kLdKeys) / kLdKeys);  // ceil((t - lo + 1) / 64)
   const int i0 = (int)((long long)tiles * rank / splits), i1 = (int)((long long)tiles * (rank + 1) / splits);
-
-  const int rc = R / 8;
-  for (int i = threadIdx.x; i < MR * rc; i += kLdThreads) {
-    const int r = i / rc, c = (i % rc) * 8;
-    const bool ok = h0 + r < p.heads;
-    const uint16_t* q = reinterpret_cast<const uint16_t*>(p.qa);
-    ld_cp16(tc_smem_u32(sq + r * lds + c), ok ? q + ((int64_t)b * p.heads + h0 + r) * R + c : q, ok);
-  }
+  const int rc = R / 8, np = (int)p.npages;
   auto fetch = [&](int i, int stage) {  // a warp per key row
 #pragma unroll
     for (int rr = 0; rr < kLdKeys / kLdWarps; rr++) {
       const int r = warp * (kLdKeys / kLdWarps) + rr;
       const int64_t j = lo + (int64_t)i * kLdKeys + r;
       const bool ok = j <= t;
-      const int64_t jj = ok ? j : t;
-      const uint16_t* src = reinterpret_cast<const uint16_t*>(__ldg(p.pages + (jj / 32) % p.npages)) + ((int64_t)b * 32 + jj % 32) * R;
+      const int jj = (int)(ok ? j : t);
+      const uint16_t* src = reinterpret_cast<const uint16_t*>(__ldg(p.pages + (jj / 32) % np)) + ((int64_t)b * 32 + jj % 32) * R;
       for (int c = lane; c < rc; c += 32) ld_cp16(tc_smem_u32(sk + ((size_t)stage * kLdKeys + r) * lds + c * 8), src + c * 8, ok);
     }
     ld_commit();
   };
+  if (i0 < i1) fetch(i0, 0);
+  else ld_commit();
+  // this warp's quarter of the queries as MMA operands
+  const int ksteps = R / 16, k0 = kq * ((ksteps + 3) / 4), k1 = min(ksteps, k0 + (ksteps + 3) / 4);
+  uint32_t qf[MT][KS][4];
+#pragma unroll
+  for (int m = 0; m < MT; m++)
+#pragma unroll
+    for (int k = 0; k < KS; k++)
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const int h = h0 + m * 16 + (lane >> 2) + (e & 1) * 8, c = (k0 + k) * 16 + (e >> 1) * 8 + (lane & 3) * 2;
+        qf[m][k][e] = (k0 + k < k1 && h < p.heads)
+                          ? __ldg(reinterpret_cast<const uint32_t*>(reinterpret_cast<const uint16_t*>(p.qa) + ((int64_t)b * p.heads + h) * R + c)) : 0u;
+      }
   for (int i = threadIdx.x; i < MR; i += kLdThreads) { sm[i] = -INFINITY; sl[i] = 0.0f; }
   float o[MT][CW][4];
 #pragma unroll
@@ -238,50 +247,58 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
   const float sc2 = p.scale * 1.4426950408889634f;
   const int cols = (krp / 8 + kLdWarps - 1) / kLdWarps;  // 8-column tiles per warp
   const int ct0 = warp * cols;
-  if (i0 < i1) fetch(i0, 0);
-  else ld_commit();
   for (int i = i0; i < i1; i++) {
     const int stage = (i - i0) & 1;
     ld_wait<0>();
     __syncthreads();  // tile i is there, and nobody still reads the other stage or the weights of tile i - 1
     if (i + 1 < i1) fetch(i + 1, stage ^ 1);
     const uint16_t* kt = sk + (size_t)stage * kLdKeys * lds;
-    {  // scores of this warp's 8 keys
-      float acc[MT][4] = {};
-      const uint32_t kb = tc_smem_u32(kt + (warp * 8 + (lane & 7)) * lds + ((lane >> 3) & 1) * 8);
-      const uint32_t qa = tc_smem_u32(sq + (lane & 15) * lds + (lane >> 4) * 8);
-#pragma unroll 4
-      for (int k = 0; k < R; k += 16) {
-        uint32_t bb[2];
-        ldm_x2(kb + k * 2, bb);
+    {
+      float acc[MT][4][4] = {};
+      const uint32_t kb = tc_smem_u32(kt + (key0 + (lane & 7) + ((lane >> 4) & 1) * 8) * lds + ((lane >> 3) & 1) * 8);
 #pragma unroll
-        for (int m = 0; m < MT; m++) {
-          uint32_t a[4];
-          ldm_x4(qa + (m * 16 * lds + k) * 2, a);
-          mma16816(acc[m], a, bb[0], bb[1]);
+      for (int k = 0; k < KS; k++) {
+        if (k0 + k < k1) {
+          uint32_t b0[4], b1[4];
+          ldm_x4(kb + (k0 + k) * 32, b0);
+          ldm_x4(kb + (16 * lds + (k0 + k) * 16) * 2, b1);
+#pragma unroll
+          for (int m = 0; m < MT; m++) {
+            mma16816(acc[m][0], qf[m][k], b0[0], b0[1]);
+            mma16816(acc[m][1], qf[m][k], b0[2], b0[3]);
+            mma16816(acc[m][2], qf[m][k], b1[0], b1[1]);
+            mma16816(acc[m][3], qf[m][k], b1[2], b1[3]);
+          }
         }
       }
-      const int key = warp * 8 + (lane & 3) * 2;
-      const int64_t left = t - (lo + (int64_t)i * kLdKeys);  // keys 0 .. left exist
 #pragma unroll
       for (int m = 0; m < MT; m++)
 #pragma unroll
-        for (int h = 0; h < 2; h++) {
-          float* d = ss + (m * 16 + (lane >> 2) + h * 8) * (kLdKeys + 4) + key;
-          d[0] = key <= left ? acc[m][2 * h] * sc2 : -INFINITY;
-          d[1] = key + 1 <= left ? acc[m][2 * h + 1] * sc2 : -INFINITY;
-        }
+        for (int n = 0; n < 4; n++)
+#pragma unroll
+          for (int h = 0; h < 2; h++)
+            *reinterpret_cast<float2*>(ss + (kq * MR + m * 16 + (lane >> 2) + h * 8) * SW + key0 + n * 8 + (lane & 3) * 2) =
+                make_float2(acc[m][n][2 * h], acc[m][n][2 * h + 1]);
     }
     __syncthreads();
+    const int left = (int)min((int64_t)kLdKeys, t - (lo + (int64_t)i * kLdKeys) + 1);  // keys 0 .. left - 1 exist
 #pragma unroll
     for (int rr = 0; rr < MR / kLdWarps; rr++) {  // softmax of this warp's heads, two keys per lane
       const int r = warp * (MR / kLdWarps) + rr;
-      const float x0 = ss[r * (kLdKeys + 4) + lane * 2], x1 = ss[r * (kLdKeys + 4) + lane * 2 + 1];
-      float mx = fmaxf(x0, x1);
+      float2 x = make_float2(0.0f, 0.0f);
+#pragma unroll
+      for (int q = 0; q < 4; q++) {
+        const float2 v = *reinterpret_cast<const float2*>(ss + (q * MR + r) * SW + lane * 2);
+        x.x += v.x;
+        x.y += v.y;
+      }
+      x.x = lane * 2 < left ? x.x * sc2 : -INFINITY;
+      x.y = lane * 2 + 1 < left ? x.y * sc2 : -INFINITY;
+      float mx = fmaxf(x.x, x.y);
 #pragma unroll
       for (int s = 16; s > 0; s >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, s));
       const float mo = sm[r], mn = fmaxf(mo, mx);  // a tile has at least one key
-      const float e0 = exp2f(x0 - mn), e1 = exp2f(x1 - mn), al = exp2f(mo - mn);
+      const float e0 = exp2f(x.x - mn), e1 = exp2f(x.y - mn), al = exp2f(mo - mn);
       const float sum = hy_warp_sum(e0 + e1);
       const uint32_t hi = ld_pack(e0, e1);
       const uint32_t low = ld_pack(e0 - __uint_as_float(hi << 16), e1 - __uint_as_float(hi & 0xffff0000u));
@@ -325,21 +342,20 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
   __syncthreads();
   tc_cluster_sync();
   float* so = reinterpret_cast<float*>(ld_smem);  // [MR][krp], over the key stages
-  for (int r = threadIdx.x; r < MR; r += kLdThreads) {
-    float mx = -INFINITY;
-    for (int c = 0; c < splits; c++) {
-      float v;
-      asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(tc_mapa(tc_smem_u32(sm + r), c)) : "memory");
-      mx = fmaxf(mx, v);
-    }
-    float tot = 0.0f;
-    for (int c = 0; c < splits; c++) {
-      float v, l;
-      asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(tc_mapa(tc_smem_u32(sm + r), c)) : "memory");
+  if (threadIdx.x < MR * 8) {  // eight lanes per head, one per CTA of the cluster
+    const int r = threadIdx.x >> 3, c = threadIdx.x & 7;
+    float m = -INFINITY, l = 0.0f;
+    if (c < splits) {
+      asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(m) : "r"(tc_mapa(tc_smem_u32(sm + r), c)) : "memory");
       asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(l) : "r"(tc_mapa(tc_smem_u32(sl + r), c)) : "memory");
-      if (l > 0.0f) tot += l * exp2f(v - mx);
     }
-    sa[r] = sl[r] > 0.0f ? exp2f(sm[r] - mx) / tot : 0.0f;
+    float mx = m;
+#pragma unroll
+    for (int x = 4; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+    float tot = l > 0.0f ? l * exp2f(m - mx) : 0.0f;
+#pragma unroll
+    for (int x = 4; x > 0; x >>= 1) tot += __shfl_xor_sync(0xffffffffu, tot, x);
+    if (c == 0) sa[r] = sl[r] > 0.0f ? exp2f(sm[r] - mx) / tot : 0.0f;
   }
   __syncthreads();
 #pragma unroll
@@ -350,78 +366,87 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
     for (int c = 0; c < CW; c++) {
       const int n = (ct0 + c) * 8 + (lane & 3) * 2;
       if (c < cols && n < krp) {
-        so[r * krp + n] = o[m][c][0] * a0;
-        so[r * krp + n + 1] = o[m][c][1] * a0;
-        so[(r + 8) * krp + n] = o[m][c][2] * a1;
-        so[(r + 8) * krp + n + 1] = o[m][c][3] * a1;
+        *reinterpret_cast<float2*>(so + r * krp + n) = make_float2(o[m][c][0] * a0, o[m][c][1] * a0);
+        *reinterpret_cast<float2*>(so + (r + 8) * krp + n) = make_float2(o[m][c][2] * a1, o[m][c][3] * a1);
       }
     }
   }
   tc_cluster_sync();
   const int nq = MR * krp / 4;
   for (int q = rank * kLdThreads + threadIdx.x; q < nq; q += splits * kLdThreads) {
-    float4 s = make_float4(0, 0, 0, 0);
-    for (int c = 0; c < splits; c++) {
-      const float4 v = tc_ld_cluster_f4(tc_mapa(tc_smem_u32(so + q * 4), c));
-      s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
-    }
+    float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+    tc_cluster_sum<1, 8>(tc_smem_u32(so + q * 4), splits, s);
     const int r = q * 4 / krp, n = q * 4 % krp;
     if (h0 + r < p.heads)
-      *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(p.ol) + ((int64_t)b * p.heads + h0 + r) * krp + n) = make_uint2(ld_pack(s.x, s.y), ld_pack(s.z, s.w));
+      *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(p.ol) + ((int64_t)b * p.heads + h0 + r) * krp + n) = make_uint2(ld_pack(s[0], s[1]), ld_pack(s[2], s[3]));
   }
   tc_cluster_sync();  // nobody leaves while its shared memory is being read
 }
 
 static size_t ld_smem_bytes(int MR, int R) {
-  return ((size_t)2 * kLdKeys * (R + 8) + (size_t)MR * (R + 8) + 2 * MR * (kLdKeys + 8)) * 2 + (size_t)MR * (kLdKeys + 4) * 4 + 3 * MR * 4;
+  return ((size_t)2 * kLdKeys * (R + 8) + 2 * MR * (kLdKeys + 8)) * 2 + (size_t)4 * MR * (kLdKeys + 4) * 4 + 3 * MR * 4;
 }
 
 bool latent_decode_serves(const TpxLatentAttn& a) {
-  if (a.f32 || a.lat || a.S != 1 || a.R % 16 || a.krp % 16 || a.krp > 512) return false;
+  if (a.f32 || a.lat || a.S != 1 || a.R % 16 || a.krp % 16 || a.krp > 512 || a.R > 640 || a.past >= (1ll << 30)) return false;
   const int MR = a.heads <= 16 ? 16 : 32;
   const size_t smem = ld_smem_bytes(MR, (int)a.R);
   return smem <= 225 * 1024 && (size_t)MR * a.krp * 4 <= (size_t)2 * kLdKeys * (a.R + 8) * 2 && (((uintptr_t)a.qa | (uintptr_t)a.ol) & 15) == 0;
 }
 
-template <int MT, int CW>
-static int latent_decode_launch(const TpxLatentAttn& a, int splits, cudaStream_t st) {
+template <int MT, int CW, int KS>
+static int latent_decode_launch(const TpxLatentAttn& a, cudaStream_t st) {
   const size_t smem = ld_smem_bytes(MT * 16, (int)a.R);
   static bool opted[16] = {};
+  static int resident[9] = {};  // clusters of each size that fit the device at once (largest shared memory of this kernel)
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 16 || !opted[dev]) {
-    TPX_CUDA_OK(cudaFuncSetAttribute(latent_decode_kernel<MT, CW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024));
+    TPX_CUDA_OK(cudaFuncSetAttribute(latent_decode_kernel<MT, CW, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024));
     if (dev >= 0 && dev < 16) opted[dev] = true;
   }
+  const int64_t groups = (a.heads + MT * 16 - 1) / (MT * 16), items = a.B * groups;
+  // keys that may be in the window (planning only; the kernel reads the count itself)
+  int64_t keys = a.npages * 32 < a.window ? a.npages * 32 : a.window;
+  if (!a.dev_len && a.past + 1 < keys) keys = a.past + 1;
+  const int64_t tiles = (keys + kLdKeys - 1) / kLdKeys;
   cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3((unsigned)(a.B * splits), (unsigned)((a.heads + MT * 16 - 1) / (MT * 16)));
   cfg.blockDim = dim3(kLdThreads);
   cfg.dynamicSmemBytes = smem;
   cfg.stream = st;
   cudaLaunchAttribute attr[2];
-  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[0].val.programmaticStreamSerializationAllowed = knobs().pdl;
-  attr[1].id = cudaLaunchAttributeClusterDimension;
-  attr[1].val.clusterDim.x = (unsigned)splits;
-  attr[1].val.clusterDim.y = 1;
-  attr[1].val.clusterDim.z = 1;
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = knobs().pdl;
   cfg.attrs = attr;
+  int splits = tiles < 8 ? (int)tiles : 8;
+  for (; splits > 1; splits--) {  // as many CTAs per sequence as run at once
+    if (items * splits > sm_count()) continue;
+    if (!resident[splits]) {
+      cfg.gridDim = dim3((unsigned)splits, 1);
+      cfg.numAttrs = 1;
+      attr[0].val.clusterDim.x = (unsigned)splits;
+      int n = 0;
+      TPX_CUDA_OK(cudaOccupancyMaxActiveClusters(&n, latent_decode_kernel<MT, CW, KS>, &cfg));
+      resident[splits] = n > 0 ? n : -1;
+    }
+    if (resident[splits] >= items) break;
+  }
+  if (splits < 1) splits = 1;
+  attr[0].val.clusterDim.x = (unsigned)splits;
+  cfg.gridDim = dim3((unsigned)(a.B * splits), (unsigned)groups);
   cfg.numAttrs = 2;
   count_launch();
-  TPX_CUDA_OK(cudaLaunchKernelEx(&cfg, latent_decode_kernel<MT, CW>, a, splits));
+  TPX_CUDA_OK(cudaLaunchKernelEx(&cfg, latent_decode_kernel<MT, CW, KS>, a, splits));
   return TPX_OK;
 }
 
 int latent_decode(const TpxLatentAttn& a, cudaStream_t st) {
-  // keys that may be in the window (planning only; the kernel reads the count itself)
-  int64_t keys = a.npages * 32 < a.window ? a.npages * 32 : a.window;
-  if (!a.dev_len && a.past + 1 < keys) keys = a.past + 1;
-  const int64_t tiles = (keys + kLdKeys - 1) / kLdKeys, groups = (a.heads + 31) / 32;
-  int splits = 1;
-  while (splits < 8 && splits * 2 <= tiles && a.B * groups * splits * 2 <= sm_count() + sm_count() / 8) splits *= 2;
-  const int cw = (int)((a.krp / 8 + kLdWarps - 1) / kLdWarps);
-  if (a.heads <= 16) return cw <= 2 ? latent_decode_launch<1, 2>(a, splits, st) : cw <= 4 ? latent_decode_launch<1, 4>(a, splits, st) : latent_decode_launch<1, 8>(a, splits, st);
-  return cw <= 2 ? latent_decode_launch<2, 2>(a, splits, st) : cw <= 4 ? latent_decode_launch<2, 4>(a, splits, st) : latent_decode_launch<2, 8>(a, splits, st);
+  const bool one = a.heads <= 16;
+  if (a.krp <= 128 && a.R <= 192) return one ? latent_decode_launch<1, 2, 3>(a, st) : latent_decode_launch<2, 2, 3>(a, st);
+  if (a.krp <= 256 && a.R <= 320) return one ? latent_decode_launch<1, 4, 5>(a, st) : latent_decode_launch<2, 4, 5>(a, st);
+  return one ? latent_decode_launch<1, 8, 10>(a, st) : latent_decode_launch<2, 8, 10>(a, st);
 }
 
 }  // namespace tpx

@@ -15,7 +15,10 @@
 //   warps 2-5: epilogue (tensor memory -> registers -> bias / activation / multiply / residual -> y)
 //
 // One CTA per SM walks a contiguous range of output tiles (the token tiles of one feature tile are neighbours, so a
-// weight tile fetched for the first of them is found in L2 by the others). Two accumulators in tensor memory: the
+// weight tile fetched for the first of them is found in L2 by the others). Up to 64 tokens the range is one of pipeline
+// stages instead (BfParams::split): every CTA streams the same number of weight bytes, and the pieces of a tile that was
+// cut are added in the order of k by the CTA that finishes last (fp32 partials and an arrival counter in the scratch; no
+// CTA waits for another). Two accumulators in tensor memory: the
 // epilogue of a tile runs under the MMAs of the next. At decode sizes the kernel is a plain stream of W at HBM rate.
 #include "tpx_hybrid.cuh"
 #include "tpx_tc_ptx.cuh"
@@ -34,7 +37,35 @@ struct BfParams {
   TcParams t;   // epilogue fields (bias, act, mul_in, res, res_scale, y, M, N, err)
   int ksteps;   // k steps of 64 (K rounded up)
   int TN, TM;   // feature tiles, token tiles
+  int split;    // 1: the CTAs share all pipeline stages of all tiles evenly; a tile cut between CTAs is put together by the last of them
   BfEx ex;
+};
+
+// The stages a CTA works on, as pieces of tiles: piece = stages [g0, g1) of one tile.
+struct BfPieces {
+  long long u, u1;
+  int ns;
+  int tile, g0, g1;
+  __device__ __forceinline__ BfPieces(const BfParams& p, int nstages) : ns(nstages) {
+    const long long T = (long long)p.TN * p.TM;
+    if (p.split) {
+      const long long U = T * ns;
+      u = blockIdx.x * U / gridDim.x;
+      u1 = (blockIdx.x + 1) * U / gridDim.x;
+    } else {
+      u = blockIdx.x * T / gridDim.x * ns;
+      u1 = (blockIdx.x + 1) * T / gridDim.x * ns;
+    }
+    tile = g0 = g1 = 0;
+  }
+  __device__ __forceinline__ bool next() {
+    if (u >= u1) return false;
+    tile = (int)(u / ns);
+    g0 = (int)(u % ns);
+    g1 = (int)min((long long)ns, g0 + (u1 - u));
+    u += g1 - g0;
+    return true;
+  }
 };
 
 // 16 consecutive tokens of output feature n; the lanes of a warp hold 32 neighbouring features
@@ -96,9 +127,8 @@ linear_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t smem_base = (tc_smem_u32(bf_smem_raw) + 1023u) & ~1023u;
-  const long long T = (long long)p.TN * p.TM;
-  const int tile0 = (int)((long long)blockIdx.x * T / gridDim.x), tile1 = (int)(((long long)blockIdx.x + 1) * T / gridDim.x);
   const int nstages = (p.ksteps + C::UK - 1) / C::UK;  // pipeline stages per tile
+  __shared__ int last_piece;
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < C::STAGES; s++) {
@@ -127,27 +157,41 @@ linear_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
   if (warp == 0) {
     // ------------------------------------------------------------ producer
     if (lane == 0) {
-      pdl_wait();  // x (and, in a chain of launches, nothing else) comes from earlier grids
+      // at decode sizes W is a model's weight, not the output of a kernel in flight: its copies for the first stages need not
+      // wait for the kernels that make x (many rows may come with a weight unpacked for the call)
+      auto copy_w = [&](int tile, int g, int s) {
+        const uint32_t st = smem_base + (uint32_t)s * C::STAGE_BYTES;
+        const uint32_t bar = tc_smem_u32(&bar_full[s]);
+        tc_mbar_expect_tx(bar, C::STAGE_BYTES);
+#pragma unroll
+        for (int u = 0; u < C::UK; u++)  // a k step beyond K reads as zeros
+          tc_tma_2d(st + u * C::A_BYTES, &tmW, (g * C::UK + u) * 64, tile / p.TM * 128, bar);
+      };
+      auto copy_x = [&](int tile, int g, int s) {
+        const uint32_t st = smem_base + (uint32_t)s * C::STAGE_BYTES;
+        const uint32_t bar = tc_smem_u32(&bar_full[s]);
+#pragma unroll
+        for (int u = 0; u < C::UK; u++)
+          tc_tma_2d(st + C::UK * C::A_BYTES + u * C::B_BYTES, &tmX, (g * C::UK + u) * 64, tile % p.TM * TOK, bar);
+      };
+      BfPieces ahead(p, nstages);
+      int pre = 0;
+      while (TOK <= 64 && pre < C::STAGES && ahead.next())
+        for (int g = ahead.g0; g < ahead.g1 && pre < C::STAGES; g++) copy_w(ahead.tile, g, pre++);
+      pdl_wait();
+      BfPieces pc(p, nstages);
       long long it = 0;
       bool dead = false;
-      for (int tile = tile0; tile < tile1 && !dead; tile++) {
-        const int tn = tile / p.TM, tm = tile % p.TM;
-        for (int g = 0; g < nstages; g++, it++) {
+      while (!dead && pc.next()) {
+        for (int g = pc.g0; g < pc.g1; g++, it++) {
           const int s = (int)(it % C::STAGES);
           if (it >= C::STAGES && !tc_wait(tc_smem_u32(&bar_empty[s]), (uint32_t)((it / C::STAGES - 1) & 1))) {
             atomicExch(p.t.err, 2u);
             dead = true;
             break;
           }
-          const uint32_t st = smem_base + (uint32_t)s * C::STAGE_BYTES;
-          const uint32_t bar = tc_smem_u32(&bar_full[s]);
-          tc_mbar_expect_tx(bar, C::STAGE_BYTES);
-#pragma unroll
-          for (int u = 0; u < C::UK; u++) {  // a k step beyond K reads as zeros
-            const int kc = (g * C::UK + u) * 64;
-            tc_tma_2d(st + u * C::A_BYTES, &tmW, kc, tn * 128, bar);
-            tc_tma_2d(st + C::UK * C::A_BYTES + u * C::B_BYTES, &tmX, kc, tm * TOK, bar);
-          }
+          if (it >= pre) copy_w(pc.tile, g, s);
+          copy_x(pc.tile, g, s);
         }
       }
     }
@@ -160,14 +204,15 @@ linear_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
       long long it = 0;
       uint32_t empty_phase = 0;  // bit b: parity to wait for on acc_empty[b]
       bool dead = false;
-      for (int tile = tile0; tile < tile1 && !dead; tile++) {
-        const int buf = (tile - tile0) & 1;
-        if (tile - tile0 >= 2) {  // the epilogue must have drained this accumulator
+      BfPieces pc(p, nstages);
+      for (int i = 0; !dead && pc.next(); i++) {
+        const int buf = i & 1;
+        if (i >= 2) {  // the epilogue must have drained this accumulator
           if (!tc_wait(tc_smem_u32(&acc_empty[buf]), (empty_phase >> buf) & 1u)) { atomicExch(p.t.err, 3u); break; }
           empty_phase ^= 1u << buf;
           tc_fence_after();
         }
-        for (int g = 0; g < nstages; g++, it++) {
+        for (int g = pc.g0; g < pc.g1; g++, it++) {
           const int s = (int)(it % C::STAGES);
           if (!tc_wait(tc_smem_u32(&bar_full[s]), (uint32_t)((it / C::STAGES) & 1))) { atomicExch(p.t.err, 4u); dead = true; break; }
           tc_fence_after();
@@ -177,7 +222,7 @@ linear_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
 #pragma unroll
             for (int j = 0; j < 4; j++) {
               bf_mma(tmem + buf * TOK, tc_smem_desc(st + u * C::A_BYTES) + (uint64_t)(2 * j),
-                     tc_smem_desc(st + C::UK * C::A_BYTES + u * C::B_BYTES) + (uint64_t)(2 * j), idesc, (g == 0 && u == 0 && j == 0) ? 0u : 1u);
+                     tc_smem_desc(st + C::UK * C::A_BYTES + u * C::B_BYTES) + (uint64_t)(2 * j), idesc, (g == pc.g0 && u == 0 && j == 0) ? 0u : 1u);
             }
           }
           tc_commit(tc_smem_u32(&bar_empty[s]));
@@ -192,33 +237,72 @@ linear_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
     const uint32_t lane_base = ((uint32_t)(sub * 32)) << 16;
     uint32_t full_phase = 0;
     pdl_wait();  // residual and multiplier inputs belong to earlier grids
-    for (int tile = tile0; tile < tile1; tile++) {
-      const int buf = (tile - tile0) & 1;
-      if (!tc_wait(tc_smem_u32(&acc_full[buf]), (full_phase >> buf) & 1u)) {
+    BfPieces pc(p, nstages);
+    const int first_tile = (int)(pc.u / nstages);
+    bool dead = false;  // a warp that gave up still meets the others at their barriers
+    for (int i = 0; pc.next(); i++) {
+      const int buf = i & 1;
+      if (!dead && !tc_wait(tc_smem_u32(&acc_full[buf]), (full_phase >> buf) & 1u)) {
         if (lane == 0) atomicExch(p.t.err, 6u);
-        break;
+        dead = true;
       }
       full_phase ^= 1u << buf;
       tc_fence_after();
-      const int tn = tile / p.TM, tm = tile % p.TM;
-      const int n = tn * 128 + sub * 32 + lane;
+      const int tn = pc.tile / p.TM, tm = pc.tile % p.TM;
+      const int nl = sub * 32 + lane, n = tn * 128 + nl;
       const int tok0 = tm * TOK;
+      const bool whole = pc.g0 == 0 && pc.g1 == nstages;
+      float* part = whole ? nullptr : p.t.partial + ((size_t)blockIdx.x * 2 + (pc.tile == first_tile ? 0 : 1)) * TOK * 128;
+      auto finish = [&](int c0, const float (&v)[16]) {
+        if (n < p.t.N && tok0 + c0 < p.t.M) {
+          const float v2[16] = {};
+          if (p.ex.on) bf_finish16_ex(p.ex, p.t.M, tok0 + c0, n, v);
+          else tc_finish16<false>(p.t, tok0 + c0, n, v, v2);
+        }
+      };
 #pragma unroll 1
-      for (int c0 = 0; c0 < TOK; c0 += 16) {
+      for (int c0 = 0; c0 < TOK && !dead; c0 += 16) {
         uint32_t a[16];
-        float v[16], v2[16];
+        float v[16];
         tc_ld_x16(tmem + lane_base + buf * TOK + c0, a);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
-        for (int j = 0; j < 16; j++) { v[j] = __uint_as_float(a[j]); v2[j] = 0.0f; }
-        if (n < p.t.N && tok0 + c0 < p.t.M) {
-          if (p.ex.on) bf_finish16_ex(p.ex, p.t.M, tok0 + c0, n, v);
-          else tc_finish16<false>(p.t, tok0 + c0, n, v, v2);
+        for (int j = 0; j < 16; j++) v[j] = __uint_as_float(a[j]);
+        if (whole) finish(c0, v);
+        else if (tok0 + c0 < p.t.M) {
+#pragma unroll
+          for (int j = 0; j < 16; j++) part[(c0 + j) * 128 + nl] = v[j];
         }
       }
       tc_fence_before();
       __syncwarp();
       if (lane == 0) tc_mbar_arrive(tc_smem_u32(&acc_empty[buf]));
+      if (!whole) {
+        // publish this piece; whoever comes last adds the tile's pieces in the order of k
+        const long long U = (long long)p.TN * p.TM * nstages, G = gridDim.x, u = (long long)pc.tile * nstages;
+        const int ca = (int)(((u + 1) * G - 1) / U), cb = (int)(((u + nstages) * G - 1) / U);
+        __threadfence();
+        asm volatile("bar.sync 1, 128;" ::: "memory");
+        if (threadIdx.x == 64) {
+          const bool last = atomicAdd(p.t.counters + pc.tile, 1u) == (unsigned)(cb - ca);
+          if (last) p.t.counters[pc.tile] = 0;
+          last_piece = last;
+        }
+        asm volatile("bar.sync 1, 128;" ::: "memory");
+        if (last_piece) {
+          __threadfence();
+#pragma unroll 1
+          for (int c0 = 0; c0 < TOK && tok0 + c0 < p.t.M; c0 += 16) {
+            float v[16] = {};
+            for (int c = ca; c <= cb; c++) {
+              const float* q = p.t.partial + ((size_t)c * 2 + ((int)(c * U / G / nstages) == pc.tile ? 0 : 1)) * TOK * 128 + c0 * 128 + nl;
+#pragma unroll
+              for (int j = 0; j < 16; j++) v[j] += __ldcg(q + j * 128);
+            }
+            finish(c0, v);
+          }
+        }
+      }
     }
   }
   tc_fence_before();
@@ -265,12 +349,30 @@ static int bf_launch(const CUtensorMap& w, const CUtensorMap& x, const BfParams&
   }
   const long long T = (long long)p.TN * p.TM;
   const int sms = sm_count();
-  TPX_CUDA_OK(launch_pdl(linear_bf16_kernel<TOK>, dim3((unsigned)(T < sms ? T : sms)), dim3(kTcThreads), C::SMEM, st, w, x, p));
+  const int grid = p.split ? p.split : (int)(T < sms ? T : sms);
+  TPX_CUDA_OK(launch_pdl(linear_bf16_kernel<TOK>, dim3((unsigned)grid), dim3(kTcThreads), C::SMEM, st, w, x, p));
   return TPX_OK;
 }
 
+// Decode sizes read every weight once: with whole tiles per CTA the rate is set by the CTA that has one tile more than the
+// others, or by the few CTAs that have any. CTAs of an even split of all stages (0: keep whole tiles).
+static int bf_split_ctas(int64_t M, int64_t N, int64_t K) {
+  if (M > 64) return 0;
+  const int64_t T = (N + 127) / 128, ns = ((K + 63) / 64 + 1) / 2, sms = sm_count();
+  if (T >= 8 * sms || T % sms == 0 || T > 16000) return 0;
+  const int64_t most = T * ns / 4;  // a CTA takes at least four stages (512 values of k)
+  const int64_t grid = most < sms ? most : sms;
+  return grid > T || T > sms ? (int)grid : 0;
+}
+static size_t bf_split_bytes(int64_t M, int grid) { return (size_t)grid * 2 * (M <= 16 ? 16 : M <= 32 ? 32 : 64) * 128 * 4; }
+
 // Tiles, tensor maps and launch for a filled epilogue.
-static int bf_run(BfParams& p, const void* w, const void* x, int64_t M, int64_t N, int64_t K, int64_t ldw, int64_t ldx, cudaStream_t st) {
+static int bf_run(BfParams& p, const void* w, const void* x, int64_t M, int64_t N, int64_t K, int64_t ldw, int64_t ldx, void* scratch,
+                  size_t scratch_bytes, cudaStream_t st) {
+  p.split = bf_split_ctas(M, N, K);
+  if (p.split && scratch_bytes < kTcCounterBytes + bf_split_bytes(M, p.split)) p.split = 0;
+  p.t.counters = reinterpret_cast<unsigned*>(scratch);
+  p.t.partial = reinterpret_cast<float*>(reinterpret_cast<unsigned char*>(scratch) + kTcCounterBytes);
   const int tok = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
   p.t.M = (int)M; p.t.N = (int)N; p.t.K = (int)K;
   p.ksteps = (int)((K + 63) / 64);
@@ -299,7 +401,7 @@ int linear_tc_ex(const TpxLinear& a, cudaStream_t st) {
   BfParams p = {};
   p.t.err = reinterpret_cast<unsigned*>(reinterpret_cast<unsigned char*>(a.scratch) + kTcCounterBytes - 4);
   p.ex = {a.bias, a.act_params, a.y, (long long)a.ldy, 1, a.out_f32, a.act, a.act_from};
-  return bf_run(p, a.w, a.x, a.M, a.N, a.K, a.ldw, a.ldx, st);
+  return bf_run(p, a.w, a.x, a.M, a.N, a.K, a.ldw, a.ldx, a.scratch, a.scratch_bytes, st);
 }
 
 }  // namespace tpx
@@ -308,7 +410,8 @@ using namespace tpx;
 
 extern "C" size_t tpx_linear_bf16_tc_scratch_bytes(int64_t M, int64_t N, int64_t K) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
-  return kTcCounterBytes;
+  const int grid = bf_split_ctas(M, N, K);
+  return kTcCounterBytes + (grid ? bf_split_bytes(M, grid) : 0);
 }
 
 extern "C" int tpx_linear_bf16_tc(const uint16_t* w, const uint16_t* x, int64_t M, int64_t N, int64_t K, const uint16_t* bias, int act,
@@ -326,5 +429,5 @@ extern "C" int tpx_linear_bf16_tc(const uint16_t* w, const uint16_t* x, int64_t 
   BfParams p = {};
   p.t.bias = bias; p.t.mul_in = mul_in; p.t.res = res; p.t.res_scale = res_scale; p.t.y = y; p.t.act = act;
   p.t.err = reinterpret_cast<unsigned*>(reinterpret_cast<unsigned char*>(scratch) + kTcCounterBytes - 4);
-  return bf_run(p, w, x, M, N, K, K, K, (cudaStream_t)stream);
+  return bf_run(p, w, x, M, N, K, K, K, scratch, scratch_bytes, (cudaStream_t)stream);
 }
