@@ -6,10 +6,12 @@
 // exponentials and square roots) are prepared by all warps into shared memory.
 // The read-outs go to `raw` in fp32; a second kernel divides each head by its root mean square and applies weight and gate.
 //
-// bf16 models with head sizes that are multiples of 8 up to 128 take delta_fast_kernel: one CTA per (sequence, head), 16 key
-// channels x CPT columns per thread (a vector read from shared memory serves CPT columns), packed two-wide fp32 arithmetic,
-// the next tokens' rows in flight (cp.async) while the current ones are worked on, output norm and gate in the same
-// kernel. Within a chunk of tokens the state is kept divided by the decay accumulated since the chunk's start, G:
+// bf16 models with head sizes that are multiples of 8 up to 128 take delta_fast_kernel: one CTA per (sequence, head),
+// DP / LPC key channels x CPT columns per thread, packed two-wide fp32 arithmetic, the next tokens' rows in flight
+// (cp.async) while the current ones are worked on, output norm and gate in the same kernel. A vector element read from
+// shared memory serves CPT columns, and shared memory gives 4 bytes per lane and cycle whatever the sharing between lanes:
+// with four columns its loads take as long as the arithmetic, with eight half as long.
+// Within a chunk of tokens the state is kept divided by the decay accumulated since the chunk's start, G:
 //   S = G s,  s <- s - (a k / G_t) q + (k / G_t) v^T,  q = (G_(t-1) k)^T s / (sum k^2 + 1e-6),
 //   o = (G_t r)^T s_(t-1) + (r . k) v - (r . a k) q
 // so that a token costs four multiply-adds per state element instead of five and reads the state once; at the chunk's end
@@ -181,61 +183,82 @@ struct DeltaFastParams {
   float eps;
 };
 
-template <int DP, int CPT, int TC>
+template <int DP, int LPC, int CPT, int TC>
 struct DfCfg {
-  static constexpr int LPC = DP / 16, THREADS = DP * LPC / CPT, NW = THREADS / 32;
-  // floats: five staged vectors per token (the values' place takes the read-outs), G, three scalars per token
-  static constexpr int STAGED = 5 * TC * DP + DP + 4 * TC;
+  static constexpr int KPT = DP / LPC, THREADS = DP * LPC / CPT, NW = THREADS / 32;
+  // floats: five staged vectors per token, the read-outs, G, three scalars per token
+  static constexpr int STAGED = 6 * TC * DP + DP + 4 * TC;
   static constexpr int RAW = TC * DP * (5 * 2 + 4);  // bytes of one raw chunk: r, k, v, a, g in bf16, w in fp32
   static constexpr size_t SMEM = STAGED * 4 + 2 * RAW;
-  static constexpr int MIN_CTAS = THREADS <= 64 ? 7 : 1;
+  static_assert(KPT % 4 == 0 && THREADS % 32 == 0 && LPC <= 32, "whole vectors and warps");
 };
 
-template <int DP, int CPT, int TC>
-__global__ void __launch_bounds__(DfCfg<DP, CPT, TC>::THREADS, DfCfg<DP, CPT, TC>::MIN_CTAS) delta_fast_kernel(DeltaFastParams p) {
-  using C = DfCfg<DP, CPT, TC>;
-  constexpr int LPC = C::LPC;
+template <int THREADS>
+__device__ __forceinline__ void df_sync() {
+  if (THREADS == 32) __syncwarp();
+  else __syncthreads();
+}
+
+// EXACT: dim == DP, so that index arithmetic is by constants
+template <int DP, int LPC, int CPT, int TC, bool EXACT>
+__global__ void __launch_bounds__(DfCfg<DP, LPC, CPT, TC>::THREADS) delta_fast_kernel(DeltaFastParams p) {
+  using C = DfCfg<DP, LPC, CPT, TC>;
+  constexpr int KV = C::KPT / 4, KP = C::KPT / 2;  // float4 vectors, channel pairs per thread
   extern __shared__ __align__(16) float df_smem[];
-  float *s_u = df_smem, *s_k = s_u + TC * DP, *s_a = s_k + TC * DP, *s_r = s_a + TC * DP, *s_v = s_r + TC * DP;
-  float* s_g = s_v + TC * DP;
-  float4* s_sc = reinterpret_cast<float4*>(s_g + DP);  // per token: 1 / (sum k^2 + 1e-6), r . k, r . (a k)
+  float *s_u = df_smem, *s_k = s_u + TC * DP, *s_a = s_k + TC * DP, *s_r = s_a + TC * DP, *s_v = s_r + TC * DP, *s_o = s_v + TC * DP;
+  float* s_g = s_o + TC * DP;
+  float4* s_sc = reinterpret_cast<float4*>(s_g + DP);  // per token: - 1 / (sum k^2 + 1e-6), r . k, r . (a k)
   unsigned char* raw = reinterpret_cast<unsigned char*>(s_sc + TC);
   pdl_trigger();
-  pdl_wait();
   const int head = blockIdx.x, b = blockIdx.y;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int l = tid % LPC, c0 = (tid / LPC) * CPT;
-  const int dim = p.dim, hd = p.H * dim;
+  const int dim = EXACT ? DP : p.dim, hd = p.H * dim;
+  constexpr int CH = DP / 32;  // channels per lane when a warp works on a token
+  float bias[CH], nw[CH];
+#pragma unroll
+  for (int i = 0; i < CH; i++) {
+    const int c = lane + 32 * i;
+    bias[i] = c < dim ? __ldg(p.a_bias + head * dim + c) : 0.0f;
+    nw[i] = c < dim ? __ldg(p.norm_w + head * dim + c) : 0.0f;
+  }
+  pdl_wait();
   const int past = p.dev_len ? *p.dev_len : p.past;
   const int first = p.start ? max(0, min(p.S, p.start[b] - past)) : 0;
+  const uint16_t* proj = p.proj + (long long)b * p.S * p.ldp + head * dim;
+  const float* wraw = p.wraw + (long long)b * p.S * hd + head * dim;
 
   auto fetch = [&](int t0, int stage) {
     unsigned char* dst = raw + stage * C::RAW;
     const int n = min(TC, p.S - t0), dc = dim / 8;  // 16-byte units per bf16 row of a head
     for (int i = tid; i < n * 5 * dc; i += C::THREADS) {
       const int c = i % dc, a = (i / dc) % 5, t = i / (dc * 5);
-      dl_cp16(dst + ((a * TC + t) * DP + c * 8) * 2, p.proj + ((long long)b * p.S + t0 + t) * p.ldp + (long long)a * hd + head * dim + c * 8);
+      dl_cp16(dst + ((a * TC + t) * DP + c * 8) * 2, proj + (long long)(t0 + t) * p.ldp + a * hd + c * 8);
     }
     for (int i = tid; i < n * 2 * dc; i += C::THREADS) {
       const int c = i % (2 * dc), t = i / (2 * dc);
-      dl_cp16(dst + 5 * TC * DP * 2 + (t * DP + c * 4) * 4, p.wraw + ((long long)b * p.S + t0 + t) * hd + head * dim + c * 4);
+      dl_cp16(dst + 5 * TC * DP * 2 + (t * DP + c * 4) * 4, wraw + (long long)(t0 + t) * hd + c * 4);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (first < p.S) fetch(first, 0);
 
-  float2 s[CPT][8];  // [column][pair of key channels]; pair i of float4 block i / 2
+  float2 s[CPT][KP];  // [column][pair of key channels]
   float* st = p.state + (long long)(b * p.H + head) * dim * dim + c0;
 #pragma unroll
-  for (int i = 0; i < 8; i++)
+  for (int i = 0; i < KP; i++)
 #pragma unroll
     for (int e = 0; e < 2; e++) {
       const int k = (i >> 1) * 4 * LPC + l * 4 + (i & 1) * 2 + e;
 #pragma unroll
-      for (int c = 0; c < CPT; c++) {
-        const float v = (k < dim && c0 + c < dim) ? st[(long long)k * dim + c] : 0.0f;
-        if (e) s[c][i].y = v;
-        else s[c][i].x = v;
+      for (int c = 0; c < CPT; c += 4) {
+        const float4 v = (k < dim && c0 + c < dim) ? *reinterpret_cast<const float4*>(st + (long long)k * dim + c) : make_float4(0, 0, 0, 0);
+        const float vv[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int d = 0; d < 4; d++) {
+          if (e) s[c + d][i].y = vv[d];
+          else s[c + d][i].x = vv[d];
+        }
       }
     }
 
@@ -243,21 +266,23 @@ __global__ void __launch_bounds__(DfCfg<DP, CPT, TC>::THREADS, DfCfg<DP, CPT, TC
   for (int t0 = first; t0 < p.S; t0 += TC, stage ^= 1) {
     const int n = min(TC, p.S - t0);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
+    df_sync<C::THREADS>();
     if (t0 + TC < p.S) fetch(t0 + TC, stage ^ 1);
     const uint16_t* rb = reinterpret_cast<const uint16_t*>(raw + stage * C::RAW);
     const float* rw = reinterpret_cast<const float*>(raw + stage * C::RAW + 5 * TC * DP * 2);
-    // decays, rates and the tokens' scalars: a warp per token
-    for (int t = warp; t < n; t += C::NW) {
+    // decays, rates and the tokens' scalars: a warp per token; tokens beyond the call's last one leave the state as it is
+#pragma unroll 2
+    for (int t = warp; t < TC; t += C::NW) {
       float k2 = 0.0f, rk = 0.0f, ra = 0.0f;
 #pragma unroll
-      for (int c = lane; c < DP; c += 32) {
+      for (int i = 0; i < CH; i++) {
+        const int c = lane + 32 * i;
         float r = 0, k = 0, v = 0, ak = 0, w = 1.0f;
-        if (c < dim) {
+        if (c < dim && t < n) {
           r = bf16_bits_to_f32(rb[(0 * TC + t) * DP + c]);
           k = bf16_bits_to_f32(rb[(1 * TC + t) * DP + c]);
           v = bf16_bits_to_f32(rb[(2 * TC + t) * DP + c]);
-          ak = dl_sigmoid(bf16_bits_to_f32(rb[(3 * TC + t) * DP + c]) + __ldg(p.a_bias + head * dim + c)) * k;
+          ak = dl_sigmoid(bf16_bits_to_f32(rb[(3 * TC + t) * DP + c]) + bias[i]) * k;
           w = __expf(-0.60653065971263342f * dl_sigmoid(rw[t * DP + c]));
         }
         k2 = fmaf(k, k, k2);
@@ -277,27 +302,29 @@ __global__ void __launch_bounds__(DfCfg<DP, CPT, TC>::THREADS, DfCfg<DP, CPT, TC
       }
       if (lane == 0) s_sc[t] = make_float4(-1.0f / (k2 + 1e-6f), rk, ra, 0.0f);
     }
-    __syncthreads();
-    // accumulated decays: a thread per channel
+    df_sync<C::THREADS>();
+    // accumulated decays: a thread per channel, all loads ahead of the stores
     for (int c = tid; c < DP; c += C::THREADS) {
+      float w[TC], k[TC], ak[TC], r[TC];
+#pragma unroll
+      for (int t = 0; t < TC; t++) { w[t] = s_u[t * DP + c]; k[t] = s_k[t * DP + c]; ak[t] = s_a[t * DP + c]; r[t] = s_r[t * DP + c]; }
       float g = 1.0f;
 #pragma unroll
       for (int t = 0; t < TC; t++) {
-        if (t < n) {
-          const float w = s_u[t * DP + c], k = s_k[t * DP + c];
-          s_u[t * DP + c] = g * k;
-          g *= w;
-          const float gi = __fdividef(1.0f, g);
-          s_k[t * DP + c] = k * gi;
-          s_a[t * DP + c] *= gi;
-          s_r[t * DP + c] *= g;
-        }
+        s_u[t * DP + c] = g * k[t];
+        g *= w[t];
+        const float gi = __fdividef(1.0f, g);
+        s_k[t * DP + c] = k[t] * gi;
+        s_a[t * DP + c] = ak[t] * gi;
+        s_r[t * DP + c] = r[t] * g;
       }
       s_g[c] = g;
     }
-    __syncthreads();
-#pragma unroll 1
-    for (int t = 0; t < n; t++) {
+    df_sync<C::THREADS>();
+    const uint32_t so = (uint32_t)__cvta_generic_to_shared(s_o);
+    constexpr int UNROLL = TC < 4 ? TC : 4;
+#pragma unroll UNROLL
+    for (int t = 0; t < TC; t++) {
       const float4* pu = reinterpret_cast<const float4*>(s_u + t * DP) + l;
       const float4* pr = reinterpret_cast<const float4*>(s_r + t * DP) + l;
       float2 qa[CPT], oa[CPT];
@@ -305,38 +332,46 @@ __global__ void __launch_bounds__(DfCfg<DP, CPT, TC>::THREADS, DfCfg<DP, CPT, TC
       for (int c = 0; c < CPT; c++) qa[c] = oa[c] = make_float2(0.0f, 0.0f);
       float v[CPT];
 #pragma unroll
-      for (int c = 0; c < CPT; c++) v[c] = s_v[t * DP + c0 + c];
+      for (int c = 0; c < CPT; c += 4) {
+        const float4 x = *reinterpret_cast<const float4*>(s_v + t * DP + c0 + c);
+        v[c] = x.x; v[c + 1] = x.y; v[c + 2] = x.z; v[c + 3] = x.w;
+      }
 #pragma unroll
-      for (int i = 0; i < 4; i++) {
-        const float4 u = pu[i * LPC], r = pr[i * LPC];
+      for (int i = 0; i < KV; i++) {
+        const float4 u = pu[i * LPC];
 #pragma unroll
         for (int c = 0; c < CPT; c++) {
           qa[c] = dl_fma2(make_float2(u.x, u.y), s[c][2 * i], qa[c]);
           qa[c] = dl_fma2(make_float2(u.z, u.w), s[c][2 * i + 1], qa[c]);
+        }
+      }
+      float q[CPT], o[CPT];
+#pragma unroll
+      for (int c = 0; c < CPT; c++) q[c] = qa[c].x + qa[c].y;
+#pragma unroll
+      for (int x = LPC / 2; x > 0; x >>= 1)
+#pragma unroll
+        for (int c = 0; c < CPT; c++) q[c] += __shfl_xor_sync(0xffffffffu, q[c], x);
+#pragma unroll
+      for (int i = 0; i < KV; i++) {  // independent of q: fills the time of the shuffles
+        const float4 r = pr[i * LPC];
+#pragma unroll
+        for (int c = 0; c < CPT; c++) {
           oa[c] = dl_fma2(make_float2(r.x, r.y), s[c][2 * i], oa[c]);
           oa[c] = dl_fma2(make_float2(r.z, r.w), s[c][2 * i + 1], oa[c]);
         }
       }
       const float4 sc = s_sc[t];
-      float q[CPT], o[CPT];
-#pragma unroll
-      for (int c = 0; c < CPT; c++) { q[c] = qa[c].x + qa[c].y; o[c] = oa[c].x + oa[c].y; }
-#pragma unroll
-      for (int x = LPC / 2; x > 0; x >>= 1)
-#pragma unroll
-        for (int c = 0; c < CPT; c++) {
-          q[c] += __shfl_xor_sync(0xffffffffu, q[c], x);
-          o[c] += __shfl_xor_sync(0xffffffffu, o[c], x);
-        }
+      const float rk = l == 0 ? sc.y : 0.0f, ra = l == 0 ? sc.z : 0.0f;  // one lane of a column adds the scalar terms
       const float4* pk = reinterpret_cast<const float4*>(s_k + t * DP) + l;
       const float4* pa = reinterpret_cast<const float4*>(s_a + t * DP) + l;
 #pragma unroll
       for (int c = 0; c < CPT; c++) {
         q[c] *= sc.x;
-        o[c] = fmaf(sc.y, v[c], fmaf(sc.z, q[c], o[c]));
+        o[c] = fmaf(rk, v[c], fmaf(ra, q[c], oa[c].x + oa[c].y));
       }
 #pragma unroll
-      for (int i = 0; i < 4; i++) {
+      for (int i = 0; i < KV; i++) {
         const float4 k = pk[i * LPC], a = pa[i * LPC];
 #pragma unroll
         for (int c = 0; c < CPT; c++) {
@@ -345,15 +380,34 @@ __global__ void __launch_bounds__(DfCfg<DP, CPT, TC>::THREADS, DfCfg<DP, CPT, TC
           s[c][2 * i + 1] = dl_fma2(make_float2(a.z, a.w), qq, dl_fma2(make_float2(k.z, k.w), vv, s[c][2 * i + 1]));
         }
       }
-      if (l == 0) {  // the column's lanes have read its value (the shuffles are behind them)
+      // sum over the column's lanes, every step leaving a lane half of its columns: lane l ends with columns l * CPT / LPC ...
+      constexpr int LEFT = CPT > LPC ? CPT / LPC : 1, SKIP = LPC > CPT ? LPC / CPT : 1;
 #pragma unroll
-        for (int c = 0; c < CPT; c++) s_v[t * DP + c0 + c] = o[c];
+      for (int x = LPC / 2, m = CPT; x > 0; x >>= 1) {
+        if (m > 1) {
+          m >>= 1;
+          const bool up = (l & x) != 0;
+#pragma unroll
+          for (int c = 0; c < CPT / 2; c++)
+            if (c < m) {
+              const float mine = up ? o[c + m] : o[c], other = up ? o[c] : o[c + m];
+              o[c] = mine + __shfl_xor_sync(0xffffffffu, other, x);
+            }
+        } else {
+          o[0] += __shfl_xor_sync(0xffffffffu, o[0], x);
+        }
       }
+      // stored without a memory clobber: nothing but the next barrier orders these against other accesses, so that the next
+      // token's loads may move ahead of them
+      if (l % SKIP == 0)
+#pragma unroll
+        for (int c = 0; c < LEFT; c++)
+          asm volatile("st.shared.f32 [%0], %1;" ::"r"(so + (uint32_t)(t * DP + c0 + l * CPT / LPC + c) * 4), "f"(o[c]));
     }
     {
       const float4* pg = reinterpret_cast<const float4*>(s_g) + l;
 #pragma unroll
-      for (int i = 0; i < 4; i++) {
+      for (int i = 0; i < KV; i++) {
         const float4 g = pg[i * LPC];
 #pragma unroll
         for (int c = 0; c < CPT; c++) {
@@ -362,50 +416,51 @@ __global__ void __launch_bounds__(DfCfg<DP, CPT, TC>::THREADS, DfCfg<DP, CPT, TC
         }
       }
     }
-    __syncthreads();
+    asm volatile("" ::: "memory");
+    df_sync<C::THREADS>();
     // output norm and gate: a warp per token
+#pragma unroll 2
     for (int t = warp; t < n; t += C::NW) {
-      float ss = 0.0f;
+      float x[CH], ss = 0.0f;
 #pragma unroll
-      for (int c = lane * 2; c < DP; c += 64) {
-        const float2 x = *reinterpret_cast<const float2*>(s_v + t * DP + c);
-        if (c < dim) ss = fmaf(x.x, x.x, fmaf(x.y, x.y, ss));
+      for (int i = 0; i < CH; i++) {
+        x[i] = lane + 32 * i < dim ? s_o[t * DP + lane + 32 * i] : 0.0f;
+        ss = fmaf(x[i], x[i], ss);
       }
       const float inv = rsqrtf(hy_warp_sum(ss) / (float)dim + p.eps);
+      uint16_t* out = p.out + ((long long)b * p.S + t0 + t) * p.ldo + head * dim;
 #pragma unroll
-      for (int c = lane * 2; c < DP; c += 64) {
-        if (c < dim) {
-          const float2 x = *reinterpret_cast<const float2*>(s_v + t * DP + c);
-          const float2 nw = __ldg(reinterpret_cast<const float2*>(p.norm_w + head * dim + c));
-          const float g0 = dl_sigmoid(bf16_bits_to_f32(rb[(4 * TC + t) * DP + c])), g1 = dl_sigmoid(bf16_bits_to_f32(rb[(4 * TC + t) * DP + c + 1]));
-          *reinterpret_cast<__nv_bfloat162*>(p.out + ((long long)b * p.S + t0 + t) * p.ldo + head * dim + c) =
-              __floats2bfloat162_rn(x.x * inv * nw.x * g0, x.y * inv * nw.y * g1);
-        }
-      }
+      for (int i = 0; i < CH; i++)
+        if (lane + 32 * i < dim)
+          out[lane + 32 * i] = f32_to_bf16_bits(x[i] * inv * nw[i] * dl_sigmoid(bf16_bits_to_f32(rb[(4 * TC + t) * DP + lane + 32 * i])));
     }
   }
 #pragma unroll
-  for (int i = 0; i < 8; i++)
+  for (int i = 0; i < KP; i++)
 #pragma unroll
     for (int e = 0; e < 2; e++) {
       const int k = (i >> 1) * 4 * LPC + l * 4 + (i & 1) * 2 + e;
 #pragma unroll
-      for (int c = 0; c < CPT; c++)
-        if (k < dim && c0 + c < dim) st[(long long)k * dim + c] = e ? s[c][i].y : s[c][i].x;
+      for (int c = 0; c < CPT; c += 4)
+        if (k < dim && c0 + c < dim)
+          *reinterpret_cast<float4*>(st + (long long)k * dim + c) =
+              e ? make_float4(s[c][i].y, s[c + 1][i].y, s[c + 2][i].y, s[c + 3][i].y) : make_float4(s[c][i].x, s[c + 1][i].x, s[c + 2][i].x, s[c + 3][i].x);
     }
 }
 
-template <int DP, int CPT, int TC>
+template <int DP, int LPC, int CPT, int TC>
 static int delta_fast_launch(const DeltaFastParams& p, int64_t B, cudaStream_t st) {
-  using C = DfCfg<DP, CPT, TC>;
+  using C = DfCfg<DP, LPC, CPT, TC>;
+  void (*k)(DeltaFastParams) = p.dim == DP ? delta_fast_kernel<DP, LPC, CPT, TC, true> : delta_fast_kernel<DP, LPC, CPT, TC, false>;
   static bool opted[16] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (C::SMEM > 48 * 1024 && (dev < 0 || dev >= 16 || !opted[dev])) {
-    TPX_CUDA_OK(cudaFuncSetAttribute(delta_fast_kernel<DP, CPT, TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
+    TPX_CUDA_OK(cudaFuncSetAttribute(delta_fast_kernel<DP, LPC, CPT, TC, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
+    TPX_CUDA_OK(cudaFuncSetAttribute(delta_fast_kernel<DP, LPC, CPT, TC, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
     if (dev >= 0 && dev < 16) opted[dev] = true;
   }
-  TPX_CUDA_OK(launch_pdl(delta_fast_kernel<DP, CPT, TC>, dim3((unsigned)p.H, (unsigned)B), dim3(C::THREADS), C::SMEM, st, p));
+  TPX_CUDA_OK(launch_pdl(k, dim3((unsigned)p.H, (unsigned)B), dim3(C::THREADS), C::SMEM, st, p));
   return TPX_OK;
 }
 
@@ -417,16 +472,15 @@ static bool delta_fast_serves(const TpxDeltaRule& a) {
 static int delta_fast(const TpxDeltaRule& a, cudaStream_t st) {
   DeltaFastParams p = {(const uint16_t*)a.proj, a.wraw, a.a_bias, a.norm_w, a.start, a.dev_len, a.state, (uint16_t*)a.out, (long long)a.ldp,
                        (long long)a.ldo, (int)a.S, (int)a.past, (int)a.heads, (int)a.dim, a.eps};
-  // columns per thread: few when the heads alone leave the machine idle (a token's latency counts), many otherwise
-  const int64_t heads = a.B * a.heads;
-  if (a.dim <= 32) return heads * 4 >= sm_count() * 16 ? delta_fast_launch<32, 2, 16>(p, a.B, st) : delta_fast_launch<32, 1, 16>(p, a.B, st);
+  // eight columns per thread and few warps per head when there are many heads, more warps per head when a token's latency counts
+  const bool many = a.B * a.heads >= (a.dim <= 64 ? 4 : 2) * sm_count();
+  if (a.dim <= 32) return a.S == 1 ? delta_fast_launch<32, 4, 4, 1>(p, a.B, st) : delta_fast_launch<32, 4, 4, 8>(p, a.B, st);
   if (a.dim <= 64) {
-    if (a.S == 1 || heads >= sm_count() * 4) return delta_fast_launch<64, 4, 8>(p, a.B, st);
-    if (heads >= sm_count() * 2) return delta_fast_launch<64, 2, 16>(p, a.B, st);
-    return delta_fast_launch<64, 1, 16>(p, a.B, st);
+    if (a.S == 1) return delta_fast_launch<64, 8, 4, 1>(p, a.B, st);
+    return many ? delta_fast_launch<64, 4, 8, 8>(p, a.B, st) : delta_fast_launch<64, 8, 4, 16>(p, a.B, st);
   }
-  if (a.S == 1 || heads >= sm_count()) return delta_fast_launch<128, 4, 8>(p, a.B, st);
-  return delta_fast_launch<128, 2, 8>(p, a.B, st);
+  if (a.S == 1) return delta_fast_launch<128, 16, 4, 1>(p, a.B, st);
+  return many ? delta_fast_launch<128, 8, 8, 8>(p, a.B, st) : delta_fast_launch<128, 16, 4, 8>(p, a.B, st);
 }
 
 template <typename T, int DP>

@@ -209,16 +209,19 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
   const int tiles = (int)((t - lo + kLdKeys) / kLdKeys);  // ceil((t - lo + 1) / 64)
   const int i0 = (int)((long long)tiles * rank / splits), i1 = (int)((long long)tiles * (rank + 1) / splits);
   const int rc = R / 8, np = (int)p.npages;
-  auto fetch = [&](int i, int stage) {  // a warp per key row
+  constexpr int ROWS = kLdKeys / kLdWarps;
+  auto fetch = [&](int i, int stage) {  // a warp per key row; lanes 0 .. ROWS - 1 first look up one row's page each
+    const int64_t j = lo + (int64_t)i * kLdKeys + warp * ROWS + (lane & (ROWS - 1));
+    const int jj = (int)(j <= t ? j : t);
+    const uint64_t mine = __ldg(p.pages + (jj / 32) % np) + ((uint64_t)b * 32 + jj % 32) * R * 2 + (j <= t ? 0u : 1u);  // odd: no such key
+    uint64_t src[ROWS];
 #pragma unroll
-    for (int rr = 0; rr < kLdKeys / kLdWarps; rr++) {
-      const int r = warp * (kLdKeys / kLdWarps) + rr;
-      const int64_t j = lo + (int64_t)i * kLdKeys + r;
-      const bool ok = j <= t;
-      const int jj = (int)(ok ? j : t);
-      const uint16_t* src = reinterpret_cast<const uint16_t*>(__ldg(p.pages + (jj / 32) % np)) + ((int64_t)b * 32 + jj % 32) * R;
-      for (int c = lane; c < rc; c += 32) ld_cp16(tc_smem_u32(sk + ((size_t)stage * kLdKeys + r) * lds + c * 8), src + c * 8, ok);
-    }
+    for (int r = 0; r < ROWS; r++) src[r] = __shfl_sync(0xffffffffu, mine, r);
+    const uint32_t dst = tc_smem_u32(sk + ((size_t)stage * kLdKeys + warp * ROWS) * lds);
+    for (int c = lane; c < rc; c += 32)
+#pragma unroll
+      for (int r = 0; r < ROWS; r++)
+        ld_cp16(dst + (r * lds + c * 8) * 2, reinterpret_cast<const void*>((src[r] & ~1ull) + c * 16), !(src[r] & 1));
     ld_commit();
   };
   if (i0 < i1) fetch(i0, 0);
@@ -282,30 +285,53 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
     }
     __syncthreads();
     const int left = (int)min((int64_t)kLdKeys, t - (lo + (int64_t)i * kLdKeys) + 1);  // keys 0 .. left - 1 exist
+    {  // softmax of this warp's MR / 8 heads, all at once: LR lanes per head, KL neighbouring keys per lane
+      constexpr int LR = 32 / (MR / kLdWarps), KL = kLdKeys / LR;
+      const int r = warp * (MR / kLdWarps) + lane / LR, k = (lane % LR) * KL;
+      float x[KL];
 #pragma unroll
-    for (int rr = 0; rr < MR / kLdWarps; rr++) {  // softmax of this warp's heads, two keys per lane
-      const int r = warp * (MR / kLdWarps) + rr;
-      float2 x = make_float2(0.0f, 0.0f);
+      for (int e = 0; e < KL; e += 4) {
+        float4 v = *reinterpret_cast<const float4*>(ss + r * SW + k + e);
 #pragma unroll
-      for (int q = 0; q < 4; q++) {
-        const float2 v = *reinterpret_cast<const float2*>(ss + (q * MR + r) * SW + lane * 2);
-        x.x += v.x;
-        x.y += v.y;
+        for (int q = 1; q < 4; q++) {
+          const float4 u = *reinterpret_cast<const float4*>(ss + (q * MR + r) * SW + k + e);
+          v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
+        }
+        x[e] = v.x; x[e + 1] = v.y; x[e + 2] = v.z; x[e + 3] = v.w;
       }
-      x.x = lane * 2 < left ? x.x * sc2 : -INFINITY;
-      x.y = lane * 2 + 1 < left ? x.y * sc2 : -INFINITY;
-      float mx = fmaxf(x.x, x.y);
+      float mx = -INFINITY;
 #pragma unroll
-      for (int s = 16; s > 0; s >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, s));
+      for (int e = 0; e < KL; e++) {
+        x[e] = k + e < left ? x[e] * sc2 : -INFINITY;
+        mx = fmaxf(mx, x[e]);
+      }
+#pragma unroll
+      for (int d = LR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
       const float mo = sm[r], mn = fmaxf(mo, mx);  // a tile has at least one key
-      const float e0 = exp2f(x.x - mn), e1 = exp2f(x.y - mn), al = exp2f(mo - mn);
-      const float sum = hy_warp_sum(e0 + e1);
-      const uint32_t hi = ld_pack(e0, e1);
-      const uint32_t low = ld_pack(e0 - __uint_as_float(hi << 16), e1 - __uint_as_float(hi & 0xffff0000u));
-      *reinterpret_cast<uint32_t*>(sp + r * (kLdKeys + 8) + lane * 2) = hi;
-      *reinterpret_cast<uint32_t*>(sp + (MR + r) * (kLdKeys + 8) + lane * 2) = low;
+      float sum = 0.0f;
+      uint32_t hi[KL / 2], low[KL / 2];
+#pragma unroll
+      for (int e = 0; e < KL; e += 2) {
+        const float e0 = exp2f(x[e] - mn), e1 = exp2f(x[e + 1] - mn);
+        sum += e0 + e1;
+        hi[e / 2] = ld_pack(e0, e1);
+        low[e / 2] = ld_pack(e0 - __uint_as_float(hi[e / 2] << 16), e1 - __uint_as_float(hi[e / 2] & 0xffff0000u));
+      }
+#pragma unroll
+      for (int d = LR / 2; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+      uint16_t* ph = sp + r * (kLdKeys + 8) + k;
+#pragma unroll
+      for (int e = 0; e < KL / 2; e += 2) {
+        *reinterpret_cast<uint2*>(ph + e * 2) = make_uint2(hi[e], hi[e + 1]);
+        *reinterpret_cast<uint2*>(ph + MR * (kLdKeys + 8) + e * 2) = make_uint2(low[e], low[e + 1]);
+      }
       __syncwarp();
-      if (lane == 0) { sm[r] = mn; sl[r] = sl[r] * al + sum; sa[r] = al; }
+      if (lane % LR == 0) {
+        const float al = exp2f(mo - mn);
+        sm[r] = mn;
+        sl[r] = sl[r] * al + sum;
+        sa[r] = al;
+      }
     }
     __syncthreads();
     // weighted sum of this warp's latent columns
