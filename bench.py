@@ -321,6 +321,144 @@ def model_decode_leg(name, shape, batch, context, steps, dev, world, rank, real_
     return out
 
 
+def _time_us(fn, n=10):
+    """Mean device time of one call of n back-to-back calls, in microseconds (CUDA events, a sleep kernel ahead of them)."""
+    import torch
+    for _ in range(3):
+        fn()
+    torch.cuda.synchronize()
+    torch.cuda._sleep(int(2e6))
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(n):
+        fn()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / n * 1e3
+
+
+def _run_model(runner, vocab, batch, context, steps, dev):
+    """Best of three prefills of batch x context random tokens, then `steps` graph-replayed decode steps behind them."""
+    import torch
+    g = torch.Generator(device="cpu").manual_seed(1234)
+    ids = torch.randint(0, vocab, (batch, context), generator=g).to(dev)
+    mask = torch.ones_like(ids)
+    runner.forward(ids[:, :64])
+    best, logits, cache = 1e30, None, None
+    for _ in range(3):
+        logits = cache = None
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record()
+        logits, cache = runner.forward(ids, mask)
+        b.record()
+        torch.cuda.synchronize()
+        best = min(best, a.elapsed_time(b))
+    timing = {}
+    sampler = ClockSampler(dev.index)
+    sampler.start()
+    runner.decode(runner._pick(logits), cache, mask, steps + 1, timing=timing)
+    torch.cuda.synchronize()
+    clocks = sampler.stop()
+    ms = timing["events"][0].elapsed_time(timing["events"][1]) / max(1, timing["steps"])
+    return {"prefill_ms": round(best, 3), "prefill_tok_s": round(batch * context / best * 1e3, 1), "ms_per_step": round(ms, 4),
+            "decode_tok_s": round(batch / ms * 1e3, 1), "clocks": clocks}
+
+
+def hybrid_ops(dev, batch, context, heads=32, width=4096, window=2048):
+    """The hybrid decoder's own kernels beside the like kernels of the Llama model, each timed alone at one layer's sizes:
+    microseconds per call and the fraction of its roofline (the slowest of bytes / copy bandwidth, tensor FLOPs / cuBLAS
+    burst, fp32 FLOPs / nominal 72.6 TFLOP/s)."""
+    import torch
+    from tpp_pytorch_extension_b200 import _lib
+    from tpp_pytorch_extension_b200._C import _hybrid_layers as HL
+    from tpp_pytorch_extension_b200._C import _fused_llm_infer as F
+    from tpp_pytorch_extension_b200._C import _tpp_attn as A
+    pk = peaks()
+    bf = lambda *s: torch.randn(*s, device=dev).to(torch.bfloat16)
+    T, out = batch * context, {}
+
+    def put(name, us, bytes_=0, tensor=0, fp32=0):
+        roof = max(bytes_ / (pk["hbm_gbs"] * 1e9), tensor / (pk["bf16_tflops"] * 1e12), fp32 / 72.6e12) * 1e6
+        out[name] = {"us": round(us, 1), "roofline_us": round(roof, 1), "frac": round(roof / us, 3)}
+
+    # residual path
+    norms = HL.Norms(1e-6, 2.0, torch.bfloat16)
+    w, conv = torch.zeros(width, device=dev), torch.randn(4, width, device=dev)
+    for name, B, S in (("prefill", batch, context), ("decode", batch, 1)):
+        x, y = torch.randn(B * S, width, device=dev), torch.randn(B * S, width, device=dev)
+        st = torch.zeros(B, 3, width, device=dev)
+        s = HL.Stream(B, S, x=x, y=y, w=w)
+        put(f"norm_conv_{name}", _time_us(lambda: norms.enter(s, conv, st, None, None, 0)), B * S * width * 14 + (B * width * 24 if S == 1 else 0))
+        xb, gam = bf(B * S, width), torch.ones(width, device=dev, dtype=torch.bfloat16)
+        put(f"llama_rmsnorm_{name}", _time_us(lambda: F.rms_norm(xb, gam, 1e-5)), B * S * width * 4)
+        del x, y, st, s, xb
+    # delta rule
+    H, d = width // 64, 64
+    for name, B, S in (("prefill", batch, context), ("decode", batch, 1), ("decode_batch64", 64, 1)):
+        TT = B * S
+        proj, wraw = bf(TT, 5 * width + 64), torch.randn(TT, width, device=dev)
+        one, zero = torch.ones(width, device=dev), torch.zeros(width, device=dev)
+        state, o = torch.zeros(B, H, d, d, device=dev), torch.empty(TT, width, dtype=torch.bfloat16, device=dev)
+
+        def delta():
+            HL._call("tpx_delta_rule", _lib.DeltaRuleStruct(
+                proj=proj.data_ptr(), wraw=wraw.data_ptr(), a_bias=zero.data_ptr(), norm_w=one.data_ptr(), state=state.data_ptr(), raw=wraw.data_ptr(),
+                out=o.data_ptr(), B=B, S=S, past=0, ldp=proj.shape[1], ldo=width, heads=H, dim=d, eps=1e-6, f32=0))
+        put(f"delta_{name}", _time_us(delta), TT * width * 16 + B * H * d * d * 8, fp32=2 * TT * width * d * 4)
+        del proj, wraw, state, o
+    # latent attention and the Llama attention
+    kvr, rot, hd, vd = 512, 64, 128, 128
+    R, win = kvr + rot, min(window, context)
+    pairs = sum(min(i + 1, win) for i in range(context))
+    gate = torch.ones(T, heads, device=dev)
+    q, kv, lat, cs = bf(T, heads * (hd + rot)), bf(T, heads * (hd + vd)), bf(T, R), torch.zeros(T, rot // 2, 2, device=dev)
+    o = torch.empty(T, heads * vd, dtype=torch.bfloat16, device=dev)
+    put("latent_attn_prefill", _time_us(lambda: HL._call("tpx_latent_prefill", _lib.LatentPrefillStruct(
+        q=q.data_ptr(), kv=kv.data_ptr(), lat=lat.data_ptr(), cos_sin=cs.data_ptr(), gate=gate.data_ptr(), out=o.data_ptr(), B=batch, S=context, L=context,
+        past=0, heads=heads, dim=hd, rot_dim=rot, vdim=vd, krp=kvr, R=R, ldq=q.shape[1], ldkv=kv.shape[1], ldo=o.shape[1], window=win, scale=0.07))),
+        2 * (q.numel() + kv.numel() + o.numel()), tensor=2 * batch * heads * pairs * (hd + rot + vd))
+    del q, kv, lat, o
+    S1 = (context + 31) // 32
+    k1, v1, q1 = bf(S1, batch, heads, 32, hd), bf(S1, batch, heads, 32, hd), bf(batch, heads, context, 1, hd)
+    put("llama_attn_prefill", _time_us(lambda: A.attention(q1, k1, v1, None, context)), 2 * (2 * k1.numel() + 2 * q1.numel()),
+        tensor=4 * batch * heads * hd * context * (context + 1) // 2)
+    q1 = bf(batch, heads, 1, 1, hd)
+    put("llama_attn_decode", _time_us(lambda: A.attention(q1, k1, v1, None, context)), 2 * 2 * batch * heads * context * hd)
+    del k1, v1, q1
+    for B in (batch, 64):
+        P = (win + 30) // 32 + 1
+        pages = bf(P, B, 32, R)
+        ptrs = torch.tensor([pages.data_ptr() + i * pages.stride(0) * 2 for i in range(P)], device=dev)
+        qa, ol = bf(B, heads, R), torch.empty(B, heads, kvr, dtype=torch.bfloat16, device=dev)
+        put(f"latent_attn_decode_batch{B}", _time_us(lambda: HL._call("tpx_latent_attn", _lib.LatentAttnStruct(
+            qa=qa.data_ptr(), pages=ptrs.data_ptr(), ol=ol.data_ptr(), B=B, S=1, L=0, past=3 * win, npages=P, heads=heads, krp=kvr, R=R, window=win,
+            scale=0.07, f32=0))), 2 * B * win * R, tensor=2 * B * heads * win * (R + kvr))
+        del pages
+    return out
+
+
+def hybrid_legs(dev, steps):
+    """Prefill and decode throughput of the hybrid decoder (bf16 random weights) beside a bf16 Llama of the same depth,
+    width, feed-forward, heads and vocabulary."""
+    import torch
+    from tpp_pytorch_extension_b200.llm import fused_dofivik_infer as FD
+    from tpp_pytorch_extension_b200.llm import fused_llama_infer as FL
+    out = {"ops": hybrid_ops(dev, 16, 2048)}
+    for layers, width, heads, ff, cells in ((8, 4096, 32, 14336, ((16, 2048), (1, 4096))), (16, 2048, 16, 8192, ((16, 1024), (1, 2048)))):
+        for name in ("dofivik", "llama"):
+            torch.cuda.empty_cache()
+            if name == "dofivik":
+                runner = FD.build_random_dofivik(FD.hybrid_shape(layers, width, heads, ff, 32000), device=dev)
+            else:
+                runner = FL.build_random_llama(FL.LlamaShape(layers, width, heads, heads, ff, 32000, max_position_embeddings=8192), "bf16", dev)
+            for batch, context in cells:
+                key = f"{layers}x{width}_batch{batch}_context{context}"
+                out.setdefault(key, {})[name] = _run_model(runner, 32000, batch, context, steps, dev)
+            del runner
+    return out
+
+
 def tp_consistency_check(dev, world):
     """Two layers of the tensor-parallel configuration's shape, same seeded weights: logits of the sharded model (this
     run's ranks) against the unsharded model built on the same GPU. max |a - b| / max |b|."""
@@ -608,6 +746,8 @@ def run_ours(args):
             legs["config5_tp_consistency"] = tp_consistency_check(dev, world)
         legs["config5_llama2_70b_mxfp4_tp"] = model_decode_leg("Llama-2-70B shape, MXFP4, tensor parallel", shape, 64, 4096, args.model_steps, dev,
                                                                world, rank, False)
+    if "hybrid" in want and world == 1:
+        legs["hybrid_decoder_bf16"] = hybrid_legs(dev, args.model_steps)
     if rank == 0:
         line["decode_models"] = legs
         print(json.dumps(line))
@@ -623,7 +763,7 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--ms", default="", help="comma-separated subset of the token counts to run (for profiler captures)")
     ap.add_argument("--legs", default="cfg3,cfg4,cfg5", help="model-level decode legs to run after the op sweep: cfg3 (Llama-2-7B shape, int8, one GPU), cfg4 (Llama-3-8B shape, one GPU), "
-                    "cfg5 (Llama-2-70B shape, tensor parallel over --gpus ranks); empty for none")
+                    "cfg5 (Llama-2-70B shape, tensor parallel over --gpus ranks), hybrid (not in the default: the hybrid decoder beside a bf16 Llama of equal size, one GPU); empty for none")
     ap.add_argument("--model-steps", type=int, default=48, help="decode steps timed in each model-level leg")
     ap.add_argument("--cfg5-layers", type=int, default=0, help="decoder layers of the 70B-shape leg (0 = all 80)")
     ap.add_argument("--min-seconds", type=float, default=1.0, help="repeat the K timed steps until this much device time was measured")

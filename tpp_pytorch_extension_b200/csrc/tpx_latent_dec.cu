@@ -32,7 +32,7 @@ __device__ __forceinline__ void ldm_x2t(uint32_t a, uint32_t (&r)[2]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(a) : "memory");
 }
 __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
@@ -248,8 +248,10 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
 #pragma unroll
       for (int e = 0; e < 4; e++) o[m][c][e] = 0.0f;
   const float sc2 = p.scale * 1.4426950408889634f;
-  const int cols = (krp / 8 + kLdWarps - 1) / kLdWarps;  // 8-column tiles per warp
+  const int cols = (krp / 16 + kLdWarps - 1) / kLdWarps * 2;  // 8-column tiles per warp, in pairs
   const int ct0 = warp * cols;
+  // No branch inside the MMA loops, so that their loads run ahead: steps and tiles this warp does not have read some other
+  // valid place, against zero queries or into accumulators that are dropped
   for (int i = i0; i < i1; i++) {
     const int stage = (i - i0) & 1;
     ld_wait<0>();
@@ -261,17 +263,16 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
       const uint32_t kb = tc_smem_u32(kt + (key0 + (lane & 7) + ((lane >> 4) & 1) * 8) * lds + ((lane >> 3) & 1) * 8);
 #pragma unroll
       for (int k = 0; k < KS; k++) {
-        if (k0 + k < k1) {
-          uint32_t b0[4], b1[4];
-          ldm_x4(kb + (k0 + k) * 32, b0);
-          ldm_x4(kb + (16 * lds + (k0 + k) * 16) * 2, b1);
+        const int kk = min(k0 + k, ksteps - 1);
+        uint32_t b0[4], b1[4];
+        ldm_x4(kb + kk * 32, b0);
+        ldm_x4(kb + (16 * lds + kk * 16) * 2, b1);
 #pragma unroll
-          for (int m = 0; m < MT; m++) {
-            mma16816(acc[m][0], qf[m][k], b0[0], b0[1]);
-            mma16816(acc[m][1], qf[m][k], b0[2], b0[3]);
-            mma16816(acc[m][2], qf[m][k], b1[0], b1[1]);
-            mma16816(acc[m][3], qf[m][k], b1[2], b1[3]);
-          }
+        for (int m = 0; m < MT; m++) {
+          mma16816(acc[m][0], qf[m][k], b0[0], b0[1]);
+          mma16816(acc[m][1], qf[m][k], b0[2], b0[3]);
+          mma16816(acc[m][2], qf[m][k], b1[0], b1[1]);
+          mma16816(acc[m][3], qf[m][k], b1[2], b1[3]);
         }
       }
 #pragma unroll
@@ -350,16 +351,17 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
         for (int term = 0; term < 2; term++)
           ldm_x4(tc_smem_u32(sp + (term * MR + m * 16 + (lane & 15)) * (kLdKeys + 8) + k + (lane >> 4) * 8), a[m][term]);
 #pragma unroll
-      for (int c = 0; c < CW; c++) {
-        if (c < cols && (ct0 + c) * 8 < krp) {
-          uint32_t bb[2];
-          ldm_x2t(tc_smem_u32(kt + (k + (lane & 15)) * lds + (ct0 + c) * 8), bb);
+      for (int c = 0; c < CW; c += 2) {
+        const int n = min((ct0 + c) * 8, krp - 16);
+        uint32_t bb[4];
+        ldm_x4t(tc_smem_u32(kt + (k + (lane & 15)) * lds + n + (lane >> 4) * 8), bb);
 #pragma unroll
-          for (int m = 0; m < MT; m++) {
-            mma16816(o[m][c], a[m][0], bb[0], bb[1]);
-            mma16816(o[m][c], a[m][1], bb[0], bb[1]);
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+          for (int term = 0; term < 2; term++) {
+            mma16816(o[m][c], a[m][term], bb[0], bb[1]);
+            mma16816(o[m][c + 1], a[m][term], bb[2], bb[3]);
           }
-        }
       }
     }
   }
@@ -472,6 +474,7 @@ int latent_decode(const TpxLatentAttn& a, cudaStream_t st) {
   const bool one = a.heads <= 16;
   if (a.krp <= 128 && a.R <= 192) return one ? latent_decode_launch<1, 2, 3>(a, st) : latent_decode_launch<2, 2, 3>(a, st);
   if (a.krp <= 256 && a.R <= 320) return one ? latent_decode_launch<1, 4, 5>(a, st) : latent_decode_launch<2, 4, 5>(a, st);
+  if (a.R <= 576) return one ? latent_decode_launch<1, 8, 9>(a, st) : latent_decode_launch<2, 8, 9>(a, st);
   return one ? latent_decode_launch<1, 8, 10>(a, st) : latent_decode_launch<2, 8, 10>(a, st);
 }
 
