@@ -413,3 +413,15 @@ def test_trace_command(cuda, tmp_path, dtype):
         if want:
             got = torch.frombuffer(bytearray(f.read_bytes()), dtype=torch.float32).view(len(want), -1)
             assert U.err(got, torch.stack(want)) < U.TOL[getattr(torch, dtype)], s["step"]
+
+
+def test_generation_command(cuda, tmp_path, capsys):
+    """The generation example on a model folder, in both types."""
+    from tpp_pytorch_extension_b200.examples import run_generation
+    cfg, w = U.model("odd", seed=8)
+    U.save_folder(tmp_path, cfg, w)
+    for dtype in ("float32", "bfloat16"):
+        run_generation.main(["--model-dir", str(tmp_path), "--dtype", dtype, "--batch-size", "2", "--input-tokens", "20", "--max-new-tokens", "12",
+                             "--num-iter", "1"])
+        line = json.loads(capsys.readouterr().out.strip().splitlines()[-1])
+        assert line["model"] == "Dofivik" and line["weight_dtype"] == dtype and line["layers"] == len(cfg["layers"])

@@ -1,7 +1,7 @@
 """Greedy generation benchmark on a random-weight Llama: the counterpart of the reference's examples/llm/run_generation.py
 (its flags --weight-dtype, --input-tokens, --max-new-tokens, --batch-size, --num-iter, --num-warmup keep their meaning;
-examples/llm/run_generation.py:36-131).  There is no checkpoint or tokenizer here: weights are seeded random values of the
-named architecture and the prompt is random token ids, so only the timing is meaningful.
+examples/llm/run_generation.py:36-131).  There is no tokenizer here: the prompt is random token ids, and unless --model-dir
+names a folder with a model, weights are seeded random values of the named architecture, so only the timing is meaningful.
 
     python -m tpp_pytorch_extension_b200.examples.run_generation --model llama3-8b --weight-dtype mxfp4 \
         --batch-size 1 --input-tokens 1024 --max-new-tokens 128
@@ -19,17 +19,20 @@ import torch
 from tpp_pytorch_extension_b200.llm import fused_llama_infer as FL
 from tpp_pytorch_extension_b200._C import _fused_llm_infer as fused_llm_cpp
 
+from tpp_pytorch_extension_b200.llm import fused_dofivik_infer as FD
 from tpp_pytorch_extension_b200.llm import fused_gptj_infer as FG
 from tpp_pytorch_extension_b200.llm import fused_opt_infer as FO
 
 MODELS = {"llama2-7b": FL.LLAMA2_7B, "llama3-8b": FL.LLAMA3_8B, "llama2-70b": FL.LLAMA2_70B,
           "opt-6.7b": FO.OPTShape(32, 4096, 32, 16384, 50272), "opt-30b": FO.OPTShape(48, 7168, 56, 28672, 50272),
-          "gptj-6b": FG.GPTJShape(28, 4096, 16, 16384, 50400, 64)}
+          "gptj-6b": FG.GPTJShape(28, 4096, 16, 16384, 50400, 64), "dofivik-8b": FD.DOFIVIK_8B}
 
 
 def main(argv=None):
     ap = argparse.ArgumentParser()
     ap.add_argument("--model", default="llama3-8b", choices=sorted(MODELS))
+    ap.add_argument("--model-dir", default="", help="folder with config.json and weights: the model class follows its config (instead of --model)")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="activation type (float32: families that run in it)")
     ap.add_argument("--weight-dtype", default="mxfp4", choices=["mxfp4", "qint8", "qint2", "bfloat16", "bfloat8", "hfloat8"])
     ap.add_argument("--batch-size", type=int, default=1)
     ap.add_argument("--input-tokens", type=int, default=1024)
@@ -52,13 +55,23 @@ def main(argv=None):
         dist.init_process_group("nccl", device_id=torch.device("cuda", local))
         fused_llm_cpp.set_pg(dist.group.WORLD)
     shape = MODELS[a.model]
+    dtype = getattr(torch, a.dtype)
     if a.layers:
         import dataclasses
-        shape = dataclasses.replace(shape, num_hidden_layers=a.layers)
+        shape = dataclasses.replace(shape, layers=shape.layers[:a.layers]) if isinstance(shape, FD.DofivikShape) else dataclasses.replace(shape, num_hidden_layers=a.layers)
     wd = {"bfloat16": "bf16"}.get(a.weight_dtype, a.weight_dtype)
     from tpp_pytorch_extension_b200.llm import llm_common
     if a.load_sharded_model:
         model = llm_common.load_sharded_model()
+    elif a.model_dir:
+        from tpp_pytorch_extension_b200.llm import model_registry
+        name = model_registry.architecture_of(a.model_dir)
+        if dtype not in model_registry.dtypes_of(name):
+            ap.error(f"{name} does not run in {a.dtype}")
+        model = model_registry.load_model(a.model_dir, dtype, "cuda", None if name == "Dofivik" else wd)
+        shape, a.model = model.shape, name
+    elif isinstance(shape, FD.DofivikShape):
+        model = FD.build_random_dofivik(shape, dtype, "cuda")
     elif isinstance(shape, FO.OPTShape):
         model = FO.build_random_opt(shape, wd, "cuda")
     elif isinstance(shape, FG.GPTJShape):
@@ -91,7 +104,7 @@ def main(argv=None):
     per_tok = (tn - t1) / steps
     if rank == 0:
         print(json.dumps({
-            "model": a.model, "weight_dtype": a.weight_dtype, "tp": world, "layers": shape.num_hidden_layers,
+            "model": a.model, "weight_dtype": a.dtype if isinstance(shape, FD.DofivikShape) else a.weight_dtype, "tp": world, "layers": shape.num_hidden_layers,
             "batch_size": a.batch_size, "input_tokens": a.input_tokens, "max_new_tokens": a.max_new_tokens,
             "graph": not a.no_graph, "first_token_ms": round(t1 * 1e3, 3), "next_token_ms": round(per_tok * 1e3, 4),
             "decode_tokens_per_s": round(a.batch_size / per_tok, 1),

@@ -85,6 +85,8 @@ def make_layer(shape, idx, w, norms, device):
 
 
 class DofivikRunner(LlamaRunner):
+    packable = False
+
     def __init__(self, shape, embed, layers, norms, final_w, head_w):
         super().__init__(shape, embed, layers, final_w, head_w, None)
         self.norms = norms

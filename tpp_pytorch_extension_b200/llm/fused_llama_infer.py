@@ -98,6 +98,7 @@ class _DecodeSession:
 
 class LlamaRunner(torch.nn.Module):
     _session = None             # cache + recorded decode step kept by generate() for its next call (_DecodeSession)
+    packable = True             # save_sharded_model can store it
     reuse_decode_graph = True   # False: every generate() call builds its cache and records its decode step anew
 
     def __init__(self, shape, embed, layers, norm_w, lm_head_w, ep):

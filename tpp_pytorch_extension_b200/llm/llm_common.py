@@ -222,6 +222,8 @@ def runner_state(runner):
     """Everything a runner holds (this rank's shard), with the weights in their quantized AND kernel layouts: loading it
     needs no quantization and no repacking."""
     import dataclasses
+    if not runner.packable:
+        raise ValueError(f"{type(runner).__name__}: this family is loaded from its model folder, not from packed shards")
     st = {"runner": type(runner).__name__, "shape": dataclasses.asdict(runner.shape), "shape_class": type(runner.shape).__name__,
           "rank": get_rank(), "size": get_size(), "layers": [_layer_state(l, getattr(runner, "ep", None) is not None) for l in runner.layers], "extra": {}}
     for k, v in vars(runner).items():
