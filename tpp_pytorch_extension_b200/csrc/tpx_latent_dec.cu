@@ -1,13 +1,14 @@
 // Decoding with latent attention in bf16: the per-head maps (keys into the query, latents into values) as small grouped
 // matrix products, and attention of all heads over the cached latents, each read once.
 //
-// Attention: a thread-block cluster per (sequence, group of 32 heads); its CTAs share the window's keys in tiles of 64.
-// A tile (64 latent rows of R values, through the page table) is staged by cp.async two deep. Eight warps: each computes
-// the part of the scores of 32 keys and all heads that a quarter of the row contributes (its slice of the queries stays in
-// registers: read from shared memory by every warp it would be the largest traffic there), then the softmax of 4 heads, then
-// the weighted sum of its eighth of the latent columns for all heads (mma.sync bf16, fp32 accumulation; a latent row is key and value at once). The weights are
-// multiplied as two bf16 terms, so that they keep their 32-bit value in effect. The CTAs of a cluster merge through
-// distributed shared memory: nothing partial goes to global memory.
+// Attention: a thread-block cluster per (sequence, group of 32 heads); its CTAs share the window's keys in tiles of 32.
+// A tile (32 latent rows of R values, through the page table) is staged by cp.async four deep. Eight warps: each computes
+// the part of the scores of 16 keys and all heads that a quarter of the row contributes (its slice of the queries stays in
+// registers: read from shared memory by every warp it would be the largest traffic there), the softmax of 4 heads, and the
+// weighted sum of its eighth of the latent columns for all heads (mma.sync bf16, fp32 accumulation; a latent row is key
+// and value at once). The scores of a tile are computed beside the weighted sum of the tile before it: two barriers per
+// tile, and independent MMAs between them. The weights are multiplied as two bf16 terms, so that they keep their 32-bit
+// value in effect. The CTAs of a cluster merge through distributed shared memory: nothing partial goes to global memory.
 #include "tpx_hybrid.cuh"
 #include "tpx_tc_ptx.cuh"
 
@@ -185,28 +186,28 @@ int latent_value_mma(const TpxLatentValue& a, cudaStream_t st) {
 }
 
 // ---------------------------------------------------------------- attention
-constexpr int kLdKeys = 64, kLdWarps = 8, kLdThreads = 256;
+constexpr int kLdKeys = 32, kLdStages = 4, kLdWarps = 8, kLdThreads = 256;
 
 // MT: 16-head tiles per CTA; CW: 8-column latent tiles per warp (krp <= CW * 64); KS: 16-value steps of a quarter row
 template <int MT, int CW, int KS>
 __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentAttn p, int splits) {
-  constexpr int MR = MT * 16, SW = kLdKeys + 4;
+  constexpr int MR = MT * 16, SW = kLdKeys + 4, PW = kLdKeys + 8;
   extern __shared__ __align__(16) unsigned char ld_smem[];
   const int R = (int)p.R, krp = (int)p.krp, lds = R + 8;
-  uint16_t* sk = reinterpret_cast<uint16_t*>(ld_smem);                 // [2][64][R + 8]
-  uint16_t* sp = sk + (size_t)2 * kLdKeys * lds;                       // [2 terms][MR][64 + 8]
-  float* ss = reinterpret_cast<float*>(sp + 2 * MR * (kLdKeys + 8));   // [4 quarters][MR][64 + 4]
+  uint16_t* sk = reinterpret_cast<uint16_t*>(ld_smem);                 // [stages][32][R + 8]
+  uint16_t* sp = sk + (size_t)kLdStages * kLdKeys * lds;               // [2 terms][MR][32 + 8]
+  float* ss = reinterpret_cast<float*>(sp + 2 * MR * (kLdKeys + 8));   // [4 quarters][MR][32 + 4]
   float* sm = ss + 4 * MR * SW;                                        // [MR] running maxima (log2 units)
   float* sl = sm + MR;                                                 // [MR] running sums
   float* sa = sl + MR;                                                 // [MR] rescaling of this tile
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int rank = blockIdx.x % splits, b = blockIdx.x / splits, h0 = blockIdx.y * MR;
-  const int kq = warp & 3, key0 = (warp >> 2) * 32;
+  const int kq = warp & 3, key0 = (warp >> 2) * 16;
   pdl_trigger();
   pdl_wait();
   const int64_t t = p.dev_len ? *p.dev_len : p.past;
   const int64_t lo = max((int64_t)(p.start ? p.start[b] : 0), t - p.window + 1);
-  const int tiles = (int)((t - lo + kLdKeys) / kLdKeys);  // ceil((t - lo + 1) / 64)
+  const int tiles = (int)((t - lo + kLdKeys) / kLdKeys);  // ceil((t - lo + 1) / 32)
   const int i0 = (int)((long long)tiles * rank / splits), i1 = (int)((long long)tiles * (rank + 1) / splits);
   const int rc = R / 8, np = (int)p.npages;
   constexpr int ROWS = kLdKeys / kLdWarps;
@@ -224,8 +225,11 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
         ld_cp16(dst + (r * lds + c * 8) * 2, reinterpret_cast<const void*>((src[r] & ~1ull) + c * 16), !(src[r] & 1));
     ld_commit();
   };
-  if (i0 < i1) fetch(i0, 0);
-  else ld_commit();
+#pragma unroll
+  for (int i = 0; i < kLdStages - 1; i++) {
+    if (i0 + i < i1) fetch(i0 + i, i);
+    else ld_commit();
+  }
   // this warp's quarter of the queries as MMA operands
   const int ksteps = R / 16, k0 = kq * ((ksteps + 3) / 4), k1 = min(ksteps, k0 + (ksteps + 3) / 4);
   uint32_t qf[MT][KS][4];
@@ -252,118 +256,127 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
   const int ct0 = warp * cols;
   // No branch inside the MMA loops, so that their loads run ahead: steps and tiles this warp does not have read some other
   // valid place, against zero queries or into accumulators that are dropped
-  for (int i = i0; i < i1; i++) {
-    const int stage = (i - i0) & 1;
-    ld_wait<0>();
-    __syncthreads();  // tile i is there, and nobody still reads the other stage or the weights of tile i - 1
-    if (i + 1 < i1) fetch(i + 1, stage ^ 1);
-    const uint16_t* kt = sk + (size_t)stage * kLdKeys * lds;
-    {
-      float acc[MT][4][4] = {};
-      const uint32_t kb = tc_smem_u32(kt + (key0 + (lane & 7) + ((lane >> 4) & 1) * 8) * lds + ((lane >> 3) & 1) * 8);
+  // scores of the warp's 16 keys and quarter row, from stage st
+  auto scores = [&](int st, float (&acc)[MT][2][4]) {
+    const uint32_t kb = tc_smem_u32(sk + ((size_t)st * kLdKeys + key0 + (lane & 7) + ((lane >> 4) & 1) * 8) * lds + ((lane >> 3) & 1) * 8);
 #pragma unroll
-      for (int k = 0; k < KS; k++) {
-        const int kk = min(k0 + k, ksteps - 1);
-        uint32_t b0[4], b1[4];
-        ldm_x4(kb + kk * 32, b0);
-        ldm_x4(kb + (16 * lds + kk * 16) * 2, b1);
+    for (int k = 0; k < KS; k++) {
+      uint32_t b[4];
+      ldm_x4(kb + min(k0 + k, ksteps - 1) * 32, b);
 #pragma unroll
-        for (int m = 0; m < MT; m++) {
-          mma16816(acc[m][0], qf[m][k], b0[0], b0[1]);
-          mma16816(acc[m][1], qf[m][k], b0[2], b0[3]);
-          mma16816(acc[m][2], qf[m][k], b1[0], b1[1]);
-          mma16816(acc[m][3], qf[m][k], b1[2], b1[3]);
-        }
+      for (int m = 0; m < MT; m++) {
+        mma16816(acc[m][0], qf[m][k], b[0], b[1]);
+        mma16816(acc[m][1], qf[m][k], b[2], b[3]);
       }
-#pragma unroll
-      for (int m = 0; m < MT; m++)
-#pragma unroll
-        for (int n = 0; n < 4; n++)
-#pragma unroll
-          for (int h = 0; h < 2; h++)
-            *reinterpret_cast<float2*>(ss + (kq * MR + m * 16 + (lane >> 2) + h * 8) * SW + key0 + n * 8 + (lane & 3) * 2) =
-                make_float2(acc[m][n][2 * h], acc[m][n][2 * h + 1]);
     }
-    __syncthreads();
+  };
+  auto put_scores = [&](const float (&acc)[MT][2][4]) {
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+      for (int n = 0; n < 2; n++)
+#pragma unroll
+        for (int h = 0; h < 2; h++)
+          *reinterpret_cast<float2*>(ss + (kq * MR + m * 16 + (lane >> 2) + h * 8) * SW + key0 + n * 8 + (lane & 3) * 2) =
+              make_float2(acc[m][n][2 * h], acc[m][n][2 * h + 1]);
+  };
+  // softmax of this warp's MR / 8 heads, all at once: LR lanes per head, KL neighbouring keys per lane
+  auto softmax = [&](int i) {
+    constexpr int LR = 32 / (MR / kLdWarps), KL = kLdKeys / LR;
     const int left = (int)min((int64_t)kLdKeys, t - (lo + (int64_t)i * kLdKeys) + 1);  // keys 0 .. left - 1 exist
-    {  // softmax of this warp's MR / 8 heads, all at once: LR lanes per head, KL neighbouring keys per lane
-      constexpr int LR = 32 / (MR / kLdWarps), KL = kLdKeys / LR;
-      const int r = warp * (MR / kLdWarps) + lane / LR, k = (lane % LR) * KL;
-      float x[KL];
+    const int r = warp * (MR / kLdWarps) + lane / LR, k = (lane % LR) * KL;
+    float x[KL] = {};
 #pragma unroll
-      for (int e = 0; e < KL; e += 4) {
-        float4 v = *reinterpret_cast<const float4*>(ss + r * SW + k + e);
-#pragma unroll
-        for (int q = 1; q < 4; q++) {
-          const float4 u = *reinterpret_cast<const float4*>(ss + (q * MR + r) * SW + k + e);
-          v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
-        }
-        x[e] = v.x; x[e + 1] = v.y; x[e + 2] = v.z; x[e + 3] = v.w;
-      }
-      float mx = -INFINITY;
-#pragma unroll
-      for (int e = 0; e < KL; e++) {
-        x[e] = k + e < left ? x[e] * sc2 : -INFINITY;
-        mx = fmaxf(mx, x[e]);
-      }
-#pragma unroll
-      for (int d = LR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-      const float mo = sm[r], mn = fmaxf(mo, mx);  // a tile has at least one key
-      float sum = 0.0f;
-      uint32_t hi[KL / 2], low[KL / 2];
+    for (int q = 0; q < 4; q++)
 #pragma unroll
       for (int e = 0; e < KL; e += 2) {
-        const float e0 = exp2f(x[e] - mn), e1 = exp2f(x[e + 1] - mn);
-        sum += e0 + e1;
-        hi[e / 2] = ld_pack(e0, e1);
-        low[e / 2] = ld_pack(e0 - __uint_as_float(hi[e / 2] << 16), e1 - __uint_as_float(hi[e / 2] & 0xffff0000u));
+        const float2 u = *reinterpret_cast<const float2*>(ss + (q * MR + r) * SW + k + e);
+        x[e] += u.x;
+        x[e + 1] += u.y;
       }
+    float mx = -INFINITY;
 #pragma unroll
-      for (int d = LR / 2; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
-      uint16_t* ph = sp + r * (kLdKeys + 8) + k;
+    for (int e = 0; e < KL; e++) {
+      x[e] = k + e < left ? x[e] * sc2 : -INFINITY;
+      mx = fmaxf(mx, x[e]);
+    }
 #pragma unroll
-      for (int e = 0; e < KL / 2; e += 2) {
-        *reinterpret_cast<uint2*>(ph + e * 2) = make_uint2(hi[e], hi[e + 1]);
-        *reinterpret_cast<uint2*>(ph + MR * (kLdKeys + 8) + e * 2) = make_uint2(low[e], low[e + 1]);
-      }
-      __syncwarp();
-      if (lane % LR == 0) {
-        const float al = exp2f(mo - mn);
-        sm[r] = mn;
-        sl[r] = sl[r] * al + sum;
-        sa[r] = al;
+    for (int d = LR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+    const float mo = sm[r], mn = fmaxf(mo, mx);  // a tile has at least one key
+    float sum = 0.0f;
+    uint16_t* ph = sp + r * PW + k;
+#pragma unroll
+    for (int e = 0; e < KL; e += 2) {
+      const float e0 = exp2f(x[e] - mn), e1 = exp2f(x[e + 1] - mn);
+      sum += e0 + e1;
+      const uint32_t hi = ld_pack(e0, e1);
+      *reinterpret_cast<uint32_t*>(ph + e) = hi;
+      *reinterpret_cast<uint32_t*>(ph + MR * PW + e) = ld_pack(e0 - __uint_as_float(hi << 16), e1 - __uint_as_float(hi & 0xffff0000u));
+    }
+#pragma unroll
+    for (int d = LR / 2; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+    __syncwarp();
+    if (lane % LR == 0) {
+      const float al = exp2f(mo - mn);
+      sm[r] = mn;
+      sl[r] = sl[r] * al + sum;
+      sa[r] = al;
+    }
+  };
+  ld_wait<kLdStages - 2>();
+  __syncthreads();
+  if (i0 < i1) {
+    float acc[MT][2][4] = {};
+    scores(0, acc);
+    put_scores(acc);
+  }
+  __syncthreads();
+  if (i0 < i1) softmax(i0);
+  // one round: the scores of tile i + 1 beside the weighted sum of tile i, then the softmax of tile i + 1
+  for (int i = i0; i < i1; i++) {
+    const int st = (i - i0) % kLdStages;
+    ld_wait<kLdStages - 3>();
+    __syncthreads();  // tile i + 1 and the weights of tile i are there, tile i - 1 is no longer read
+    if (i + kLdStages - 1 < i1) fetch(i + kLdStages - 1, (st + kLdStages - 1) % kLdStages);
+    else ld_commit();
+    float acc[MT][2][4] = {};
+    scores((st + 1) % kLdStages, acc);  // behind the last tile: of whatever is there, not used
+    bool scale = false;
+#pragma unroll
+    for (int m = 0; m < MT; m++) scale |= sa[m * 16 + (lane >> 2)] != 1.0f || sa[m * 16 + (lane >> 2) + 8] != 1.0f;
+    if (__any_sync(0xffffffffu, scale)) {
+#pragma unroll
+      for (int m = 0; m < MT; m++) {
+        const float a0 = sa[m * 16 + (lane >> 2)], a1 = sa[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+        for (int c = 0; c < CW; c++) { o[m][c][0] *= a0; o[m][c][1] *= a0; o[m][c][2] *= a1; o[m][c][3] *= a1; }
       }
     }
-    __syncthreads();
-    // weighted sum of this warp's latent columns
-#pragma unroll
-    for (int m = 0; m < MT; m++) {
-      const float a0 = sa[m * 16 + (lane >> 2)], a1 = sa[m * 16 + (lane >> 2) + 8];
-#pragma unroll
-      for (int c = 0; c < CW; c++) { o[m][c][0] *= a0; o[m][c][1] *= a0; o[m][c][2] *= a1; o[m][c][3] *= a1; }
-    }
+    const uint16_t* kt = sk + (size_t)st * kLdKeys * lds;
 #pragma unroll
     for (int k = 0; k < kLdKeys; k += 16) {
       uint32_t a[MT][2][4];
 #pragma unroll
       for (int m = 0; m < MT; m++)
 #pragma unroll
-        for (int term = 0; term < 2; term++)
-          ldm_x4(tc_smem_u32(sp + (term * MR + m * 16 + (lane & 15)) * (kLdKeys + 8) + k + (lane >> 4) * 8), a[m][term]);
+        for (int term = 0; term < 2; term++) ldm_x4(tc_smem_u32(sp + (term * MR + m * 16 + (lane & 15)) * PW + k + (lane >> 4) * 8), a[m][term]);
 #pragma unroll
       for (int c = 0; c < CW; c += 2) {
         const int n = min((ct0 + c) * 8, krp - 16);
         uint32_t bb[4];
         ldm_x4t(tc_smem_u32(kt + (k + (lane & 15)) * lds + n + (lane >> 4) * 8), bb);
 #pragma unroll
-        for (int m = 0; m < MT; m++)
+        for (int term = 0; term < 2; term++)
 #pragma unroll
-          for (int term = 0; term < 2; term++) {
+          for (int m = 0; m < MT; m++) {
             mma16816(o[m][c], a[m][term], bb[0], bb[1]);
             mma16816(o[m][c + 1], a[m][term], bb[2], bb[3]);
           }
       }
     }
+    put_scores(acc);
+    __syncthreads();
+    if (i + 1 < i1) softmax(i + 1);
   }
   // merge: every CTA scales its sums to the cluster's maximum and total, then adds up its share of the columns
   ld_wait<0>();
@@ -412,14 +425,14 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
 }
 
 static size_t ld_smem_bytes(int MR, int R) {
-  return ((size_t)2 * kLdKeys * (R + 8) + 2 * MR * (kLdKeys + 8)) * 2 + (size_t)4 * MR * (kLdKeys + 4) * 4 + 3 * MR * 4;
+  return ((size_t)kLdStages * kLdKeys * (R + 8) + 2 * MR * (kLdKeys + 8)) * 2 + (size_t)4 * MR * (kLdKeys + 4) * 4 + 3 * MR * 4;
 }
 
 bool latent_decode_serves(const TpxLatentAttn& a) {
   if (a.f32 || a.lat || a.S != 1 || a.R % 16 || a.krp % 16 || a.krp > 512 || a.R > 640 || a.past >= (1ll << 30)) return false;
   const int MR = a.heads <= 16 ? 16 : 32;
   const size_t smem = ld_smem_bytes(MR, (int)a.R);
-  return smem <= 225 * 1024 && (size_t)MR * a.krp * 4 <= (size_t)2 * kLdKeys * (a.R + 8) * 2 && (((uintptr_t)a.qa | (uintptr_t)a.ol) & 15) == 0;
+  return smem <= 225 * 1024 && (size_t)MR * a.krp * 4 <= (size_t)kLdStages * kLdKeys * (a.R + 8) * 2 && (((uintptr_t)a.qa | (uintptr_t)a.ol) & 15) == 0;
 }
 
 template <int MT, int CW, int KS>
