@@ -409,7 +409,7 @@ def hybrid_ops(dev, batch, context, heads=32, width=4096, window=2048):
         del proj, wraw, state, o
     # latent attention and the Llama attention
     kvr, rot, hd, vd = 512, 64, 128, 128
-    R, win = kvr + rot, min(window, context)
+    R, win = kvr + rot + 8, min(window, context)
     pairs = sum(min(i + 1, win) for i in range(context))
     gate = torch.ones(T, heads, device=dev)
     q, kv, lat, cs = bf(T, heads * (hd + rot)), bf(T, heads * (hd + vd)), bf(T, R), torch.zeros(T, rot // 2, 2, device=dev)
@@ -433,7 +433,7 @@ def hybrid_ops(dev, batch, context, heads=32, width=4096, window=2048):
         qa, ol = bf(B, heads, R), torch.empty(B, heads, kvr, dtype=torch.bfloat16, device=dev)
         put(f"latent_attn_decode_batch{B}", _time_us(lambda: HL._call("tpx_latent_attn", _lib.LatentAttnStruct(
             qa=qa.data_ptr(), pages=ptrs.data_ptr(), ol=ol.data_ptr(), B=B, S=1, L=0, past=3 * win, npages=P, heads=heads, krp=kvr, R=R, window=win,
-            scale=0.07, f32=0))), 2 * B * win * R, tensor=2 * B * heads * win * (R + kvr))
+            scale=0.07, f32=0))), 2 * B * win * (kvr + rot), tensor=2 * B * heads * win * (2 * kvr + rot))
         del pages
     return out
 

@@ -70,7 +70,7 @@ int tpx_postnorm_final(const TpxPostnormFinal* a, void* stream);
 int tpx_argmax_f32(const float* x, int64_t rows, int64_t n, int64_t* out, void* stream);
 
 /* Rows of the latent cache: R elements = kv_rank latent values, zeros up to `krp`, rot_dim rotated key values, zeros up to
- * R. The cache is `npages` pages of [B][32][R]; token t lives in page (t / 32) mod npages, so that a windowed layer reuses
+ * R. With krp and the rotated part padded to multiples of 16 and R 8 more than their sum, the tensor-core decode serves. The cache is `npages` pages of [B][32][R]; token t lives in page (t / 32) mod npages, so that a windowed layer reuses
  * its pages. A call with several tokens also has them in `lat` [B][L][R], whose row i holds token past - (L - S) + i. */
 typedef struct {
   const float* proj; /* [T][ldp] fp32: q_rank query latents, then (own_kv) kv_rank + rot_dim, then heads gate inputs */
@@ -105,6 +105,8 @@ int tpx_latent_absorb(const TpxLatentAbsorb* a, void* stream);
 
 /* Softmax attention in the latent space: ol[T][heads][krp] = sum_j p_j c_j over the keys j of the token's window
  * (window tokens including itself), from the pages (lat == NULL, S == 1) or from lat [B][L][R]. */
+/* The copies of the bf16 single-token kernel are waited for with a bound: tpx_latent_decode_status reads (and clears) the
+ * code of a wait that gave up. */
 typedef struct {
   const void *qa, *lat;
   const uint64_t* pages;
@@ -115,6 +117,7 @@ typedef struct {
   int f32;
 } TpxLatentAttn;
 int tpx_latent_attn(const TpxLatentAttn* a, void* stream);
+int tpx_latent_decode_status(void* stream, unsigned* status_host);
 
 /* out[T][ldo] = gate * (W_uv(head) ol), head by head; w_uv [heads * vdim][krp]; columns beyond heads * vdim set to zero. */
 typedef struct {

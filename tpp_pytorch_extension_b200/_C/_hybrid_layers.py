@@ -126,7 +126,7 @@ class LatentAttention:
         vec = lambda t: t.to(device, torch.float32).contiguous()
         self.q_rank = w["dq"].shape[0]
         self.krp = round_up(kv_rank, 16)
-        self.R = self.krp + round_up(rot_dim, 16)
+        self.R = self.krp + round_up(rot_dim, 16) + 8  # 16 mod 32 bytes: the rows of a page start in different banks
         down = [w["dq"]] + ([w["dkv"]] if source is None else []) + [w["g"]]
         self.down = pad_matrix(mat(torch.cat(down, 0)))
         self.q_norm = vec(w["dq_norm"])

@@ -76,6 +76,7 @@ _SIGS = {
     "tpx_latent_gather": (c_int, [c_vp] + [c_i64] * 6 + [c_vp, c_int, c_vp]),
     "tpx_latent_absorb": (c_int, [c_vp, c_vp]),
     "tpx_latent_attn": (c_int, [c_vp, c_vp]),
+    "tpx_latent_decode_status": (c_int, [c_vp, ctypes.POINTER(ctypes.c_uint)]),
     "tpx_latent_value": (c_int, [c_vp, c_vp]),
     "tpx_latent_prefill_serves": (c_int, [c_i64] * 3),
     "tpx_latent_prefill": (c_int, [c_vp, c_vp]),
@@ -210,12 +211,12 @@ def assert_no_kernel_error(sync=True):
         code = inst.error_code()
         if code:
             raise TpxError(f"the peer-memory all-reduce gave up waiting for rank {code - 1}")
-    for name in ("tpx_attention_tc_status", "tpx_latent_tc_status"):
+    for name in ("tpx_attention_tc_status", "tpx_latent_tc_status", "tpx_latent_decode_status"):
         if _lib is not None and hasattr(_lib, name) and torch.cuda.is_available():
             st = ctypes.c_uint(0)
             check(getattr(_lib, name)(stream(), ctypes.byref(st)))
             if st.value:
-                raise TpxError(f"a prefill attention kernel gave up on a bounded wait ({name}: code {st.value})")
+                raise TpxError(f"an attention kernel gave up on a bounded wait ({name}: code {st.value})")
 
 
 _scratch = {}

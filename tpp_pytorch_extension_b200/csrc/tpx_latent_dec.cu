@@ -2,7 +2,9 @@
 // matrix products, and attention of all heads over the cached latents, each read once.
 //
 // Attention: a thread-block cluster per (sequence, group of 32 heads); its CTAs share the window's keys in tiles of 32.
-// A tile (32 latent rows of R values, through the page table) is staged by cp.async four deep. Eight warps: each computes
+// A tile is a page's 32 rows of one sequence, contiguous in the cache: one bulk copy, four of them in flight (a copy per
+// row, or cp.async, spent a quarter of the kernel's time on requests). The cache rows carry 8 elements of padding so that
+// rows lie in different banks as they are. Rows of a page outside the window are cleared after the copy. Eight warps: each computes
 // the part of the scores of 16 keys and all heads that a quarter of the row contributes (its slice of the queries stays in
 // registers: read from shared memory by every warp it would be the largest traffic there), the softmax of 4 heads, and the
 // weighted sum of its eighth of the latent columns for all heads (mma.sync bf16, fp32 accumulation; a latent row is key
@@ -186,6 +188,7 @@ int latent_value_mma(const TpxLatentValue& a, cudaStream_t st) {
 }
 
 // ---------------------------------------------------------------- attention
+static __device__ unsigned g_latent_dec_err;  // set when a bounded wait gave up; read and cleared by tpx_latent_decode_status
 constexpr int kLdKeys = 32, kLdStages = 4, kLdWarps = 8, kLdThreads = 256;
 
 // MT: 16-head tiles per CTA; CW: 8-column latent tiles per warp (krp <= CW * 64); KS: 16-value steps of a quarter row
@@ -193,8 +196,8 @@ template <int MT, int CW, int KS>
 __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentAttn p, int splits) {
   constexpr int MR = MT * 16, SW = kLdKeys + 4, PW = kLdKeys + 8;
   extern __shared__ __align__(16) unsigned char ld_smem[];
-  const int R = (int)p.R, krp = (int)p.krp, lds = R + 8;
-  uint16_t* sk = reinterpret_cast<uint16_t*>(ld_smem);                 // [stages][32][R + 8]
+  const int R = (int)p.R, krp = (int)p.krp, lds = R;
+  uint16_t* sk = reinterpret_cast<uint16_t*>(ld_smem);                 // [stages][32][R]
   uint16_t* sp = sk + (size_t)kLdStages * kLdKeys * lds;               // [2 terms][MR][32 + 8]
   float* ss = reinterpret_cast<float*>(sp + 2 * MR * (kLdKeys + 8));   // [4 quarters][MR][32 + 4]
   float* sm = ss + 4 * MR * SW;                                        // [MR] running maxima (log2 units)
@@ -203,35 +206,46 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int rank = blockIdx.x % splits, b = blockIdx.x / splits, h0 = blockIdx.y * MR;
   const int kq = warp & 3, key0 = (warp >> 2) * 16;
+  __shared__ __align__(8) unsigned long long full[kLdStages];
   pdl_trigger();
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kLdStages; i++) tc_mbar_init(tc_smem_u32(&full[i]), 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  }
+  __syncthreads();
   pdl_wait();
   const int64_t t = p.dev_len ? *p.dev_len : p.past;
   const int64_t lo = max((int64_t)(p.start ? p.start[b] : 0), t - p.window + 1);
-  const int tiles = (int)((t - lo + kLdKeys) / kLdKeys);  // ceil((t - lo + 1) / 32)
+  const int blk0 = (int)(lo / kLdKeys), tiles = (int)(t / kLdKeys) - blk0 + 1;  // tile i: the keys of page blk0 + i
   const int i0 = (int)((long long)tiles * rank / splits), i1 = (int)((long long)tiles * (rank + 1) / splits);
-  const int rc = R / 8, np = (int)p.npages;
-  constexpr int ROWS = kLdKeys / kLdWarps;
-  auto fetch = [&](int i, int stage) {  // a warp per key row; lanes 0 .. ROWS - 1 first look up one row's page each
-    const int64_t j = lo + (int64_t)i * kLdKeys + warp * ROWS + (lane & (ROWS - 1));
-    const int jj = (int)(j <= t ? j : t);
-    const uint64_t mine = __ldg(p.pages + (jj / 32) % np) + ((uint64_t)b * 32 + jj % 32) * R * 2 + (j <= t ? 0u : 1u);  // odd: no such key
-    uint64_t src[ROWS];
-#pragma unroll
-    for (int r = 0; r < ROWS; r++) src[r] = __shfl_sync(0xffffffffu, mine, r);
-    const uint32_t dst = tc_smem_u32(sk + ((size_t)stage * kLdKeys + warp * ROWS) * lds);
-    for (int c = lane; c < rc; c += 32)
-#pragma unroll
-      for (int r = 0; r < ROWS; r++)
-        ld_cp16(dst + (r * lds + c * 8) * 2, reinterpret_cast<const void*>((src[r] & ~1ull) + c * 16), !(src[r] & 1));
-    ld_commit();
+  const int np = (int)p.npages;
+  auto fetch = [&](int i) {  // one thread
+    const uint32_t bar = tc_smem_u32(&full[(i - i0) % kLdStages]);
+    const uint16_t* src = reinterpret_cast<const uint16_t*>(__ldg(p.pages + (blk0 + i) % np)) + (int64_t)b * kLdKeys * R;
+    tc_mbar_expect_tx(bar, (uint32_t)(kLdKeys * R * 2));
+    tc_bulk_g2s(tc_smem_u32(sk + (size_t)((i - i0) % kLdStages) * kLdKeys * lds), src, (uint32_t)(kLdKeys * R * 2), bar);
   };
-#pragma unroll
-  for (int i = 0; i < kLdStages - 1; i++) {
-    if (i0 + i < i1) fetch(i0 + i, i);
-    else ld_commit();
-  }
+  bool dead = false;
+  auto arrived = [&](int i) {  // tile i is in shared memory
+    if (!dead && !tc_wait(tc_smem_u32(&full[(i - i0) % kLdStages]), (uint32_t)(((i - i0) / kLdStages) & 1))) {
+      dead = true;
+      atomicExch(&g_latent_dec_err, 1u);
+    }
+    const int64_t k0 = (int64_t)(blk0 + i) * kLdKeys;
+    if (k0 < lo || k0 + kLdKeys - 1 > t) {  // the first and the last page: what lies outside may be anything
+      uint16_t* kt = sk + (size_t)((i - i0) % kLdStages) * kLdKeys * lds;
+      for (int q = threadIdx.x; q < kLdKeys * (R / 8); q += kLdThreads) {
+        const int64_t key = k0 + q / (R / 8);
+        if (key < lo || key > t) *reinterpret_cast<uint4*>(kt + q * 8) = make_uint4(0, 0, 0, 0);
+      }
+      __syncthreads();
+    }
+  };
+  if (threadIdx.x == 0)
+    for (int i = i0; i < min(i1, i0 + kLdStages - 1); i++) fetch(i);
   // this warp's quarter of the queries as MMA operands
-  const int ksteps = R / 16, k0 = kq * ((ksteps + 3) / 4), k1 = min(ksteps, k0 + (ksteps + 3) / 4);
+  const int ksteps = (R - 8) / 16, k0 = kq * ((ksteps + 3) / 4), k1 = min(ksteps, k0 + (ksteps + 3) / 4);
   uint32_t qf[MT][KS][4];
 #pragma unroll
   for (int m = 0; m < MT; m++)
@@ -283,7 +297,8 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
   // softmax of this warp's MR / 8 heads, all at once: LR lanes per head, KL neighbouring keys per lane
   auto softmax = [&](int i) {
     constexpr int LR = 32 / (MR / kLdWarps), KL = kLdKeys / LR;
-    const int left = (int)min((int64_t)kLdKeys, t - (lo + (int64_t)i * kLdKeys) + 1);  // keys 0 .. left - 1 exist
+    const int64_t key0 = (int64_t)(blk0 + i) * kLdKeys;
+    const int from = (int)max((int64_t)0, lo - key0), left = (int)min((int64_t)kLdKeys, t - key0 + 1);  // keys from .. left - 1 count
     const int r = warp * (MR / kLdWarps) + lane / LR, k = (lane % LR) * KL;
     float x[KL] = {};
 #pragma unroll
@@ -297,7 +312,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
     float mx = -INFINITY;
 #pragma unroll
     for (int e = 0; e < KL; e++) {
-      x[e] = k + e < left ? x[e] * sc2 : -INFINITY;
+      x[e] = k + e >= from && k + e < left ? x[e] * sc2 : -INFINITY;
       mx = fmaxf(mx, x[e]);
     }
 #pragma unroll
@@ -323,9 +338,8 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
       sa[r] = al;
     }
   };
-  ld_wait<kLdStages - 2>();
-  __syncthreads();
   if (i0 < i1) {
+    arrived(i0);
     float acc[MT][2][4] = {};
     scores(0, acc);
     put_scores(acc);
@@ -335,10 +349,9 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
   // one round: the scores of tile i + 1 beside the weighted sum of tile i, then the softmax of tile i + 1
   for (int i = i0; i < i1; i++) {
     const int st = (i - i0) % kLdStages;
-    ld_wait<kLdStages - 3>();
-    __syncthreads();  // tile i + 1 and the weights of tile i are there, tile i - 1 is no longer read
-    if (i + kLdStages - 1 < i1) fetch(i + kLdStages - 1, (st + kLdStages - 1) % kLdStages);
-    else ld_commit();
+    __syncthreads();  // the weights of tile i are there, tile i - 1 is no longer read
+    if (threadIdx.x == 0 && i + kLdStages - 1 < i1) fetch(i + kLdStages - 1);
+    if (i + 1 < i1) arrived(i + 1);
     float acc[MT][2][4] = {};
     scores((st + 1) % kLdStages, acc);  // behind the last tile: of whatever is there, not used
     bool scale = false;
@@ -379,7 +392,6 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
     if (i + 1 < i1) softmax(i + 1);
   }
   // merge: every CTA scales its sums to the cluster's maximum and total, then adds up its share of the columns
-  ld_wait<0>();
   __syncthreads();
   tc_cluster_sync();
   float* so = reinterpret_cast<float*>(ld_smem);  // [MR][krp], over the key stages
@@ -425,14 +437,14 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(TpxLatentA
 }
 
 static size_t ld_smem_bytes(int MR, int R) {
-  return ((size_t)kLdStages * kLdKeys * (R + 8) + 2 * MR * (kLdKeys + 8)) * 2 + (size_t)4 * MR * (kLdKeys + 4) * 4 + 3 * MR * 4;
+  return ((size_t)kLdStages * kLdKeys * R + 2 * MR * (kLdKeys + 8)) * 2 + (size_t)4 * MR * (kLdKeys + 4) * 4 + 3 * MR * 4;
 }
 
 bool latent_decode_serves(const TpxLatentAttn& a) {
-  if (a.f32 || a.lat || a.S != 1 || a.R % 16 || a.krp % 16 || a.krp > 512 || a.R > 640 || a.past >= (1ll << 30)) return false;
+  if (a.f32 || a.lat || a.S != 1 || a.R % 16 != 8 || a.krp % 16 || a.krp > 512 || a.R > 648 || a.past >= (1ll << 30)) return false;
   const int MR = a.heads <= 16 ? 16 : 32;
   const size_t smem = ld_smem_bytes(MR, (int)a.R);
-  return smem <= 225 * 1024 && (size_t)MR * a.krp * 4 <= (size_t)kLdStages * kLdKeys * (a.R + 8) * 2 && (((uintptr_t)a.qa | (uintptr_t)a.ol) & 15) == 0;
+  return smem <= 225 * 1024 && (size_t)MR * a.krp * 4 <= (size_t)kLdStages * kLdKeys * a.R * 2 && (((uintptr_t)a.qa | (uintptr_t)a.ol) & 15) == 0;
 }
 
 template <int MT, int CW, int KS>
@@ -451,6 +463,7 @@ static int latent_decode_launch(const TpxLatentAttn& a, cudaStream_t st) {
   int64_t keys = a.npages * 32 < a.window ? a.npages * 32 : a.window;
   if (!a.dev_len && a.past + 1 < keys) keys = a.past + 1;
   const int64_t tiles = (keys + kLdKeys - 1) / kLdKeys;
+  TPX_REQUIRE(a.npages < (1ll << 30), TPX_ERR_UNSUPPORTED, "latent decode: page table too long");
   cudaLaunchConfig_t cfg = {};
   cfg.blockDim = dim3(kLdThreads);
   cfg.dynamicSmemBytes = smem;
@@ -485,10 +498,25 @@ static int latent_decode_launch(const TpxLatentAttn& a, cudaStream_t st) {
 
 int latent_decode(const TpxLatentAttn& a, cudaStream_t st) {
   const bool one = a.heads <= 16;
-  if (a.krp <= 128 && a.R <= 192) return one ? latent_decode_launch<1, 2, 3>(a, st) : latent_decode_launch<2, 2, 3>(a, st);
-  if (a.krp <= 256 && a.R <= 320) return one ? latent_decode_launch<1, 4, 5>(a, st) : latent_decode_launch<2, 4, 5>(a, st);
-  if (a.R <= 576) return one ? latent_decode_launch<1, 8, 9>(a, st) : latent_decode_launch<2, 8, 9>(a, st);
+  if (a.krp <= 128 && a.R <= 200) return one ? latent_decode_launch<1, 2, 3>(a, st) : latent_decode_launch<2, 2, 3>(a, st);
+  if (a.krp <= 256 && a.R <= 328) return one ? latent_decode_launch<1, 4, 5>(a, st) : latent_decode_launch<2, 4, 5>(a, st);
+  if (a.R <= 584) return one ? latent_decode_launch<1, 8, 9>(a, st) : latent_decode_launch<2, 8, 9>(a, st);
   return one ? latent_decode_launch<1, 8, 10>(a, st) : latent_decode_launch<2, 8, 10>(a, st);
 }
 
 }  // namespace tpx
+
+using namespace tpx;
+
+extern "C" int tpx_latent_decode_status(void* stream, unsigned* status_host) {
+  TPX_REQUIRE(status_host, TPX_ERR_ARG, "latent_decode_status: null pointer");
+  static void* ptrs[64] = {};
+  int dev = 0;
+  TPX_CUDA_OK(cudaGetDevice(&dev));
+  TPX_REQUIRE(dev >= 0 && dev < 64, TPX_ERR_UNSUPPORTED, "latent_decode_status: device index %d out of range", dev);
+  if (!ptrs[dev]) TPX_CUDA_OK(cudaGetSymbolAddress(&ptrs[dev], g_latent_dec_err));
+  TPX_CUDA_OK(cudaMemcpyAsync(status_host, ptrs[dev], 4, cudaMemcpyDeviceToHost, (cudaStream_t)stream));
+  TPX_CUDA_OK(cudaMemsetAsync(ptrs[dev], 0, 4, (cudaStream_t)stream));
+  TPX_CUDA_OK(cudaStreamSynchronize((cudaStream_t)stream));
+  return TPX_OK;
+}
