@@ -281,10 +281,11 @@ def test_unequal_batch_against_each_alone(cuda, dtype, name):
         lg, cache = r.forward(ids, None, None, cache)
 
 
-def test_storage_used_again(cuda):
+@pytest.mark.parametrize("dtype,name", [(torch.float32, "mixed"), (torch.bfloat16, "mixed"), (torch.bfloat16, "wide")])
+def test_storage_used_again(cuda, dtype, name):
     """A cache whose pages and states held another request gives what a fresh one gives, also when the pages hold NaN."""
-    cfg, w = U.model("mixed", seed=6)
-    r = U.runner_of(cfg, w, torch.float32)
+    cfg, w = U.model(name, seed=6)
+    r = U.runner_of(cfg, w, dtype)
     r.only_last_logit = False
     a, b = U.tokens(cfg, 150, 1), U.tokens(cfg, 90, 2)
     want = P.forward(cfg, w, b)
@@ -300,7 +301,7 @@ def test_storage_used_again(cuda):
         for t in range(40, 90):
             lg, _ = r.forward(torch.tensor([[b[t]]], device=cuda), None, None, cache)
             got.append(lg[0])
-        assert U.err(torch.cat(got, 0), want) < U.TOL[torch.float32]
+        assert U.err(torch.cat(got, 0), want) < U.TOL[dtype]
 
 
 def greedy(cfg, w, prompt, n):

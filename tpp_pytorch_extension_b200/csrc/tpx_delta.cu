@@ -191,6 +191,7 @@ struct DfCfg {
   static constexpr int RAW = TC * DP * (5 * 2 + 4);  // bytes of one raw chunk: r, k, v, a, g in bf16, w in fp32
   static constexpr size_t SMEM = STAGED * 4 + 2 * RAW;
   static_assert(KPT % 4 == 0 && THREADS % 32 == 0 && LPC <= 32, "whole vectors and warps");
+  static_assert(CPT == 2 || CPT % 4 == 0, "columns in pairs or fours");
 };
 
 template <int THREADS>
@@ -250,15 +251,22 @@ __global__ void __launch_bounds__(DfCfg<DP, LPC, CPT, TC>::THREADS) delta_fast_k
 #pragma unroll
     for (int e = 0; e < 2; e++) {
       const int k = (i >> 1) * 4 * LPC + l * 4 + (i & 1) * 2 + e;
+      if constexpr (CPT % 4 == 0) {
 #pragma unroll
-      for (int c = 0; c < CPT; c += 4) {
-        const float4 v = (k < dim && c0 + c < dim) ? *reinterpret_cast<const float4*>(st + (long long)k * dim + c) : make_float4(0, 0, 0, 0);
-        const float vv[4] = {v.x, v.y, v.z, v.w};
+        for (int c = 0; c < CPT; c += 4) {
+          const float4 v = (k < dim && c0 + c < dim) ? *reinterpret_cast<const float4*>(st + (long long)k * dim + c) : make_float4(0, 0, 0, 0);
+          const float vv[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
-        for (int d = 0; d < 4; d++) {
-          if (e) s[c + d][i].y = vv[d];
-          else s[c + d][i].x = vv[d];
+          for (int d = 0; d < 4; d++) {
+            if (e) s[c + d][i].y = vv[d];
+            else s[c + d][i].x = vv[d];
+          }
         }
+      } else {
+        const int c = 0;
+        const float2 v = (k < dim && c0 + c < dim) ? *reinterpret_cast<const float2*>(st + (long long)k * dim + c) : make_float2(0, 0);
+        if (e) { s[c][i].y = v.x; s[c + 1][i].y = v.y; }
+        else { s[c][i].x = v.x; s[c + 1][i].x = v.y; }
       }
     }
 
@@ -331,10 +339,15 @@ __global__ void __launch_bounds__(DfCfg<DP, LPC, CPT, TC>::THREADS) delta_fast_k
 #pragma unroll
       for (int c = 0; c < CPT; c++) qa[c] = oa[c] = make_float2(0.0f, 0.0f);
       float v[CPT];
+      if constexpr (CPT % 4 == 0) {
 #pragma unroll
-      for (int c = 0; c < CPT; c += 4) {
-        const float4 x = *reinterpret_cast<const float4*>(s_v + t * DP + c0 + c);
-        v[c] = x.x; v[c + 1] = x.y; v[c + 2] = x.z; v[c + 3] = x.w;
+        for (int c = 0; c < CPT; c += 4) {
+          const float4 x = *reinterpret_cast<const float4*>(s_v + t * DP + c0 + c);
+          v[c] = x.x; v[c + 1] = x.y; v[c + 2] = x.z; v[c + 3] = x.w;
+        }
+      } else {
+        const float2 x = *reinterpret_cast<const float2*>(s_v + t * DP + c0);
+        v[0] = x.x; v[1] = x.y;
       }
 #pragma unroll
       for (int i = 0; i < KV; i++) {
@@ -440,11 +453,17 @@ __global__ void __launch_bounds__(DfCfg<DP, LPC, CPT, TC>::THREADS) delta_fast_k
 #pragma unroll
     for (int e = 0; e < 2; e++) {
       const int k = (i >> 1) * 4 * LPC + l * 4 + (i & 1) * 2 + e;
+      if constexpr (CPT % 4 == 0) {
 #pragma unroll
-      for (int c = 0; c < CPT; c += 4)
-        if (k < dim && c0 + c < dim)
-          *reinterpret_cast<float4*>(st + (long long)k * dim + c) =
-              e ? make_float4(s[c][i].y, s[c + 1][i].y, s[c + 2][i].y, s[c + 3][i].y) : make_float4(s[c][i].x, s[c + 1][i].x, s[c + 2][i].x, s[c + 3][i].x);
+        for (int c = 0; c < CPT; c += 4)
+          if (k < dim && c0 + c < dim)
+            *reinterpret_cast<float4*>(st + (long long)k * dim + c) =
+                e ? make_float4(s[c][i].y, s[c + 1][i].y, s[c + 2][i].y, s[c + 3][i].y) : make_float4(s[c][i].x, s[c + 1][i].x, s[c + 2][i].x, s[c + 3][i].x);
+      } else {
+        const int c = 0;
+        if (k < dim && c0 < dim)
+          *reinterpret_cast<float2*>(st + (long long)k * dim + c) = e ? make_float2(s[c][i].y, s[c + 1][i].y) : make_float2(s[c][i].x, s[c + 1][i].x);
+      }
     }
 }
 
@@ -477,10 +496,11 @@ static int delta_fast(const TpxDeltaRule& a, cudaStream_t st) {
   if (a.dim <= 32) return a.S == 1 ? delta_fast_launch<32, 4, 4, 1>(p, a.B, st) : delta_fast_launch<32, 4, 4, 8>(p, a.B, st);
   if (a.dim <= 64) {
     if (a.S == 1) return delta_fast_launch<64, 8, 4, 1>(p, a.B, st);
-    return many ? delta_fast_launch<64, 4, 8, 8>(p, a.B, st) : delta_fast_launch<64, 8, 4, 16>(p, a.B, st);
+    if (many) return delta_fast_launch<64, 4, 8, 8>(p, a.B, st);
+    return a.B * a.heads > sm_count() ? delta_fast_launch<64, 8, 4, 16>(p, a.B, st) : delta_fast_launch<64, 8, 2, 16>(p, a.B, st);
   }
   if (a.S == 1) return delta_fast_launch<128, 16, 4, 1>(p, a.B, st);
-  return many ? delta_fast_launch<128, 8, 8, 8>(p, a.B, st) : delta_fast_launch<128, 16, 4, 8>(p, a.B, st);
+  return many ? delta_fast_launch<128, 8, 8, 8>(p, a.B, st) : delta_fast_launch<128, 8, 4, 8>(p, a.B, st);
 }
 
 template <typename T, int DP>
