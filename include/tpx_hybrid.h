@@ -1,7 +1,7 @@
 /*
- * tpx_b200 — C ABI of the hybrid decoder's mechanisms: a linear with row strides, 32-bit or bf16 operands and 32-bit
+ * tpx_b200 — C ABI of the hybrid decoders' mechanisms: a linear with row strides, 32-bit or bf16 operands and 32-bit
  * results; the post-norm residual sum with its input convolution; latent attention over a windowed page cache; the
- * generalized delta rule. Conventions are those of tpx_b200.h. `f32` fields select the activation type of a call: 0 =
+ * generalized delta rule; the Dynamic Tanh stream; gated linear attention; chunked differential attention. Conventions are those of tpx_b200.h. `f32` fields select the activation type of a call: 0 =
  * bf16 tensors, 1 = fp32 tensors (all arithmetic in true 32-bit). The residual stream, norms, gates, rotation angles,
  * scores and recurrent state are 32-bit in both.
  *
@@ -21,11 +21,18 @@ extern "C" {
 
 /* further activations of tpx_linear: tanh; xIELU with act_params = {softplus(p), 1/2 + softplus(q)}:
  * z > 0: a0 z^2 + z/2, else a1 (e^z - 1 - z) + z/2 */
-enum { TPX_ACT_TANH = 4, TPX_ACT_XIELU = 5 };
+enum { TPX_ACT_TANH = 4, TPX_ACT_XIELU = 5, TPX_ACT_CLAMPED_GLU = 6 };
 
 /* y[M][N] = act(x[M][K] . w[N][K]^T + bias[N]); the activation applies to columns n >= act_from. Leading dimensions in
  * elements. bf16 operands run on the tcgen05 kernel and need K, ldx, ldw multiples of 8 and 16-byte aligned bases; fp32
- * operands run on the 32-bit kernel and need nothing. scratch as tpx_linear_bf16_tc. */
+ * operands run on the 32-bit kernel and need nothing. scratch as tpx_linear_bf16_tc.
+ *
+ * TPX_ACT_CLAMPED_GLU: the columns from act_from (even) on are pairs (g, u) of one gated unit each, which gives
+ * z[M][(N - act_from) / 2] = g' s(1.702 g') (u' + 1) with s the logistic function, g' = min(g, limit) and u' clamped to
+ * +-limit; y has the columns before act_from only.
+ *
+ * x_out != NULL: the result is added to a residual stream and normed for its next reader, nothing goes to y:
+ * x_out = res + result + add (fp32 rows of ldr; add [N] may be NULL), h = tanh(norm_alpha x_out) norm_w + norm_b. */
 typedef struct {
   const void *w, *x;
   const float *bias, *act_params; /* NULL: none */
@@ -34,6 +41,12 @@ typedef struct {
   int f32, out_f32, act, act_from;
   void* scratch;
   size_t scratch_bytes;
+  void* z;
+  const float *res, *add, *norm_w, *norm_b;
+  float* x_out;
+  void* h;
+  int64_t ldz, ldr, ldh;
+  float limit, norm_alpha;
 } TpxLinear;
 int tpx_linear(const TpxLinear* a, void* stream);
 
@@ -162,6 +175,67 @@ typedef struct {
   int f32;
 } TpxDeltaRule;
 int tpx_delta_rule(const TpxDeltaRule* a, void* stream);
+
+/* The residual stream at its start, or between two layers without a linear in front: x_out[n][D] = scale embed[ids] (ids !=
+ * NULL) or x, plus add [D] (may be NULL); h[n][ldh] = tanh(alpha x_out) w + b, columns from D on zero. x_out may be NULL. */
+typedef struct {
+  const int64_t* ids;
+  const void* embed; /* [vocab][D] */
+  const float *x, *add, *w, *b;
+  float* x_out;
+  void* h;
+  int64_t n, D, ldh;
+  float scale, alpha;
+  int f32;
+} TpxDyt;
+int tpx_dyt(const TpxDyt* a, void* stream);
+
+/* Gated linear attention over S tokens: per head and token S <- diag(w) S + k v^T, o = S^T (q / sqrt(dim)), with the decay
+ * w = s(z)^(1/tau) per key channel, s the logistic function; then o over its root mean square, times norm_w [vdim], times
+ * g s(g). proj [T][ldp] holds q and k (heads * dim columns each), v and g (heads * vdim each) from the columns given on. z is
+ * read from zraw [T][heads * dim], or, for a single token that tpx_gla_token_serves, computed as a2 [heads * dim][lda2] times
+ * the `rank` columns of proj from a1_col on, plus a2_bias (zraw == NULL). state [B][heads][dim][vdim] fp32 is updated in
+ * place; raw [T][heads * vdim] fp32 is working space; out rows have ldo elements. Padding rows of out become zero. */
+typedef struct {
+  const void* proj;
+  const float* zraw;
+  const void* a2;
+  const float *a2_bias, *norm_w;
+  const int32_t *start, *dev_len;
+  float *state, *raw;
+  void* out;
+  int64_t B, S, past, ldp, ldo, lda2, rank, heads, dim, vdim, q_col, k_col, v_col, g_col, a1_col;
+  float tau, eps;
+  int f32;
+} TpxGla;
+int tpx_gla_token_serves(int64_t dim, int64_t vdim);
+int tpx_gla(const TpxGla* a, void* stream);
+
+/* Chunked differential attention with capped scores. proj [T][ldp] holds heads x (2 x dim) queries, kv_heads x (2 x dim) keys
+ * and kv_heads x vdim values from the columns given on. A token at position i (leading padding not counted) sees the tokens of
+ * its chunk, positions i / chunk * chunk .. i. Per map m: softmax of softcap tanh(scale q_m . k_m / softcap); with the maps'
+ * outputs a1 and a2, o = a1 - lambda a2, then o over its root mean square, times `mult`. Query head h reads key / value head
+ * h / (heads / kv_heads).
+ *
+ * The cache is `npages` pages of [B][kv_heads][32][R]: token t in page (t / 32) mod npages; a row holds map 1's key, map 2's key
+ * (each padded with zeros to dp = dim rounded up to 16), the value, and zeros up to R, which is 2 dp + vdim rounded up to 16, plus 8.
+ * The call appends its tokens. Several tokens also need the earlier rows that are still in reach: back = min(past, chunk - 1) of
+ * them (L = back + S); `live` [B][L][kv_heads][R] is working space for them and the new rows, which may be NULL when back is 0
+ * and tpx_diff_prefill_serves. The waits inside the bf16 kernels are bounded: tpx_diff_status reads (and clears) the code of
+ * one that gave up. */
+typedef struct {
+  const void* proj;
+  const uint64_t* pages;
+  void* live;
+  const int32_t *start, *dev_len;
+  void* out;
+  int64_t B, S, L, past, npages, ldp, ldo, heads, kv_heads, dim, vdim, R, chunk, q_col, k_col, v_col;
+  float scale, softcap, lambda, mult, eps;
+  int f32;
+} TpxDiffAttn;
+int tpx_diff_prefill_serves(int64_t dim, int64_t vdim, float softcap);
+int tpx_diff_attn(const TpxDiffAttn* a, void* stream);
+int tpx_diff_status(void* stream, unsigned* status_host);
 
 #ifdef __cplusplus
 }

@@ -1,5 +1,6 @@
 """Layers of hybrid decoders on the kernels of include/tpx_hybrid.h: latent attention with a sliding window, the
-generalized delta rule and a dense feed-forward, each behind a post-norm residual with an input convolution.
+generalized delta rule and a dense feed-forward, each behind a post-norm residual with an input convolution; gated linear
+attention and chunked differential attention beside a clamped gated feed-forward in parallel layers.
 
 Activations are bf16 or, for a model built in float32, true 32-bit throughout; the residual stream, norms, gates, angles,
 scores and recurrent states are 32-bit in both. Weight matrices are stored with their rows padded to whole 16-byte units
@@ -12,7 +13,7 @@ from .. import _lib
 from .. import _timers
 from ._fused_llm_infer import bf16_linear_scratch
 
-ACT = {None: 0, "gelu": 1, "silu": 2, "relu": 3, "tanh": 4, "xielu": 5}
+ACT = {None: 0, "gelu": 1, "silu": 2, "relu": 3, "tanh": 4, "xielu": 5, "clamped_glu": 6}
 
 
 def round_up(n, m):
@@ -35,20 +36,41 @@ def _call(name, st):
         _lib.check(rc)
 
 
-def linear(x, w, bias=None, act=None, act_from=0, act_params=None, out_f32=False):
-    """act(x . w^T + bias): x [M, >= K] and w [N, K] of one type (bf16 or fp32), rows possibly strided; bias and act_params
-    fp32; the activation applies to output columns from act_from on. Result bf16 unless the operands are fp32 or out_f32."""
-    f32 = w.dtype == torch.float32
+def _linear_call(x, w, y, bias=None, **fields):
     M, (N, K) = x.shape[0], w.shape
-    y = torch.empty((M, N), dtype=torch.float32 if (f32 or out_f32) else torch.bfloat16, device=x.device)
     if x.dtype != w.dtype or x.shape[1] != K:
         raise _lib.TpxError(f"linear: input {tuple(x.shape)} {x.dtype} does not fit the weight {tuple(w.shape)} {w.dtype}")
     sc = _lib.scratch(bf16_linear_scratch(M), x.device)
     _call("tpx_linear", _lib.LinearStruct(
-        w=w.data_ptr(), x=x.data_ptr(), bias=_lib.ptr(bias), act_params=_lib.ptr(act_params), y=y.data_ptr(), M=M, N=N, K=K,
-        ldw=w.stride(0), ldx=x.stride(0), ldy=N, f32=int(f32), out_f32=int(y.dtype == torch.float32), act=ACT[act], act_from=act_from,
-        scratch=sc.data_ptr(), scratch_bytes=sc.numel()))
+        w=w.data_ptr(), x=x.data_ptr(), bias=_lib.ptr(bias), y=_lib.ptr(y), M=M, N=N, K=K, ldw=w.stride(0), ldx=x.stride(0),
+        ldy=y.stride(0) if y is not None else 0, f32=int(w.dtype == torch.float32), out_f32=int(y is not None and y.dtype == torch.float32),
+        scratch=sc.data_ptr(), scratch_bytes=sc.numel(), **fields))
+
+
+def linear(x, w, bias=None, act=None, act_from=0, act_params=None, out_f32=False):
+    """act(x . w^T + bias): x [M, >= K] and w [N, K] of one type (bf16 or fp32), rows possibly strided; bias and act_params
+    fp32; the activation applies to output columns from act_from on. Result bf16 unless the operands are fp32 or out_f32."""
+    y = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32 if (w.dtype == torch.float32 or out_f32) else torch.bfloat16, device=x.device)
+    _linear_call(x, w, y, bias, act=ACT[act], act_from=act_from, act_params=_lib.ptr(act_params))
     return y
+
+
+def linear_glu(x, w, bias, act_from, limit, z):
+    """x . w^T + bias whose columns from act_from on are (gate, up) pairs of clamped gated units: these go to z [M, units]
+    (rows possibly strided), the columns before them are returned."""
+    y = torch.empty((x.shape[0], act_from), dtype=w.dtype, device=x.device)
+    _linear_call(x, w, y, bias, act=ACT["clamped_glu"], act_from=act_from, limit=limit, z=z.data_ptr(), ldz=z.stride(0))
+    return y
+
+
+def linear_residual(x, w, res, add, norm):
+    """The residual stream behind a linear and the norm of its next reader, norm = (alpha, w, b): x_out = res + x . w^T + add
+    (fp32 [M, N]; add may be None) and tanh(alpha x_out) w + b in the type of x."""
+    alpha, nw, nb = norm
+    x_out, h = torch.empty_like(res), torch.empty(res.shape, dtype=x.dtype, device=x.device)
+    _linear_call(x, w, None, res=res.data_ptr(), add=_lib.ptr(add), norm_w=nw.data_ptr(), norm_b=nb.data_ptr(), norm_alpha=alpha,
+                 x_out=x_out.data_ptr(), h=h.data_ptr(), ldr=res.stride(0), ldh=h.stride(0))
+    return x_out, h
 
 
 def argmax_rows_f32(x):
@@ -301,4 +323,182 @@ class HybridDecoderLayer:
             s = Stream(B, S, x=x, y=y, w=self.norm2)
         if dev_len is None:
             lc.offset += S
+        return [s]
+
+
+def dynamic_tanh(norm, dtype, ids=None, embed=None, scale=1.0, x=None, add=None):
+    """The stream at its start, scale embed[ids], or a given x [n, D], plus add; returns (stream fp32, its norm in `dtype`)."""
+    alpha, w, b = norm
+    src = ids if ids is not None else x
+    n, D = (ids.numel(), embed.shape[1]) if ids is not None else x.shape
+    x_out, h = torch.empty((n, D), dtype=torch.float32, device=src.device), torch.empty((n, round_up(D, 8)), dtype=dtype, device=src.device)
+    _call("tpx_dyt", _lib.DytStruct(ids=_lib.ptr(ids), embed=_lib.ptr(embed) if ids is not None else None, x=_lib.ptr(x), add=_lib.ptr(add), w=w.data_ptr(),
+                                    b=b.data_ptr(), x_out=x_out.data_ptr(), h=h.data_ptr(), n=n, D=D, ldh=h.shape[1], scale=scale, alpha=alpha,
+                                    f32=int(dtype == torch.float32)))
+    return x_out, h
+
+
+def _sections(parts):
+    """Row blocks of one linear, each padded to whole 16-byte units: (their rows stacked, first row of each)."""
+    at, cols = 0, []
+    for p in parts:
+        cols.append(at)
+        at += round_up(p.shape[0], 8)
+    return torch.cat([pad_matrix(p) for p in parts], 0), cols
+
+
+class GatedLinearAttention:
+    """Linear attention with a decay per key channel from a low-rank map.
+
+    weights: q, k [heads * dim, D], v, g [heads * vdim, D], a1 [rank, D], a2 [heads * dim, rank], a2_bias, norm [vdim],
+    o [D, heads * vdim]. The projections are rows `self.rows` of the layer's input linear."""
+
+    def __init__(self, w, heads, dim, vdim, tau, eps, dtype, device):
+        self.heads, self.dim, self.vdim, self.tau, self.eps, self.dtype = heads, dim, vdim, float(tau), float(eps), dtype
+        mat = lambda t: t.to(device, dtype)
+        vec = lambda t: t.to(device, torch.float32).contiguous()
+        for n, rows in (("q", dim), ("k", dim), ("v", vdim), ("g", vdim), ("a2", dim)):
+            if w[n].shape[0] != heads * rows:
+                raise ValueError(f"gated linear attention: '{n}' has {w[n].shape[0]} rows, {heads} heads of {rows} are configured")
+        self.rows, self.cols = _sections([mat(w[n]) for n in ("q", "k", "v", "g", "a1")])
+        self.rows_bias = None
+        self.rank = w["a1"].shape[0]
+        self.a2, self.a2_bias, self.norm = pad_matrix(mat(w["a2"]), 1, 8), vec(w["a2_bias"]), vec(w["norm"])
+        self.o = pad_matrix(mat(w["o"]), 1, 8)
+        self.fused_decay = bool(_lib.lib().tpx_gla_token_serves(dim, vdim))
+
+    def state(self, lc, B, device):
+        return lc.state("gla", (B, self.heads, self.dim, self.vdim), device)
+
+    def reserve(self, lc, B, tokens, device):
+        self.state(lc, B, device)
+
+    def forward(self, proj, out, lc, cache, step):
+        """proj [T, >= rows]: the input linear's result; out [T, heads * vdim]: columns of the output linear's input."""
+        B, S, T = step.B, step.S, step.B * step.S
+        dev, (q, k, v, g, a1) = proj.device, self.cols
+        zraw = raw = None
+        if S > 1 or not self.fused_decay:
+            zraw = linear(proj[:, a1:a1 + self.a2.shape[1]], self.a2, bias=self.a2_bias, out_f32=True)
+            raw = torch.empty((T, self.heads * self.vdim), dtype=torch.float32, device=dev)
+        _call("tpx_gla", _lib.GlaStruct(
+            proj=proj.data_ptr(), zraw=_lib.ptr(zraw), a2=self.a2.data_ptr(), a2_bias=self.a2_bias.data_ptr(), norm_w=self.norm.data_ptr(),
+            start=_lib.ptr(step.start), dev_len=_lib.ptr(step.dev_len), state=self.state(lc, B, dev).data_ptr(), raw=_lib.ptr(raw), out=out.data_ptr(),
+            B=B, S=S, past=step.past, ldp=proj.stride(0), ldo=out.stride(0), lda2=self.a2.stride(0), rank=self.rank, heads=self.heads, dim=self.dim,
+            vdim=self.vdim, q_col=q, k_col=k, v_col=v, g_col=g, a1_col=a1, tau=self.tau, eps=self.eps, f32=int(self.dtype == torch.float32)))
+
+
+class DifferentialAttention:
+    """Differential attention (two maps per head over shared values) with capped scores, within chunks of the sequence.
+
+    weights: q [heads * 2 * dim, D], k [kv_heads * 2 * dim, D], v [kv_heads * vdim, D] and their biases q_bias, k_bias, v_bias,
+    lq1, lk1, lq2, lk2 [dim], o [D, heads * vdim]. diff: the constant part of lambda."""
+
+    def __init__(self, w, heads, kv_heads, dim, vdim, chunk, scale, softcap, diff, eps, dtype, device):
+        self.heads, self.kv_heads, self.dim, self.vdim, self.eps, self.dtype = heads, kv_heads, dim, vdim, float(eps), dtype
+        self.chunk, self.scale, self.softcap = min(int(chunk), 1 << 29), float(scale), float(softcap)
+        mat = lambda t: t.to(device, dtype)
+        if heads % kv_heads:
+            raise ValueError(f"differential attention: {heads} heads cannot share {kv_heads} key/value heads evenly")
+        for n, rows in (("q", heads * 2 * dim), ("k", kv_heads * 2 * dim), ("v", kv_heads * vdim)):
+            if w[n].shape[0] != rows:
+                raise ValueError(f"differential attention: '{n}' has {w[n].shape[0]} rows, {rows} are configured")
+        self.rows, self.cols = _sections([mat(w[n]) for n in ("q", "k", "v")])
+        self.rows_bias = torch.cat([pad_vector(w[n + "_bias"].to(device, torch.float32)) for n in ("q", "k", "v")])
+        l = {n: w[n].double() for n in ("lq1", "lk1", "lq2", "lk2")}
+        self.lam = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum()) + diff)
+        self.mult = 1.0 - float(diff)
+        self.o = pad_matrix(mat(w["o"]), 1, 8)
+        self.R = 2 * round_up(dim, 16) + round_up(vdim, 16) + 8  # both keys, the value; 16 mod 32 bytes: rows start in different banks
+        self.direct = dtype == torch.bfloat16 and bool(_lib.lib().tpx_diff_prefill_serves(dim, vdim, self.softcap))
+
+    def reserve(self, lc, B, tokens, device):
+        lc.ensure_pages((B, self.kv_heads, 32, self.R), tokens, self.chunk, self.dtype, device)
+
+    def forward(self, proj, out, lc, cache, step):
+        B, S, past = step.B, step.S, step.past
+        dev, (q, k, v) = proj.device, self.cols
+        if step.dev_len is None:
+            self.reserve(lc, B, S, dev)
+        live, L = None, S
+        if S > 1:  # the cached tokens still in reach come in front of the call's own
+            L += min(past, self.chunk - 1)
+            if L > S or not self.direct:
+                live = torch.empty((B, L, self.kv_heads, self.R), dtype=self.dtype, device=dev)
+        _call("tpx_diff_attn", _lib.DiffAttnStruct(
+            proj=proj.data_ptr(), pages=lc.ptrs.data_ptr(), live=_lib.ptr(live), start=_lib.ptr(step.start), dev_len=_lib.ptr(step.dev_len),
+            out=out.data_ptr(), B=B, S=S, L=L, past=past, npages=lc.pages(), ldp=proj.stride(0), ldo=out.stride(0), heads=self.heads,
+            kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, R=self.R, chunk=self.chunk, q_col=q, k_col=k, v_col=v, scale=self.scale,
+            softcap=self.softcap, lam=self.lam, mult=self.mult, eps=self.eps, f32=int(self.dtype == torch.float32)))
+
+
+class NormedStream:
+    """The residual stream between two parallel layers: x [T, D] fp32 and h, its norm for the next reader."""
+
+    def __init__(self, B, S, x, h):
+        self.B, self.S, self.x, self.h = B, S, x, h
+
+    @property
+    def shape(self):
+        return (self.B, self.S, self.x.shape[-1])
+
+
+class ParallelBlock:
+    """Weights of a layer whose mixer and feed-forward read one normed input and are added together: one linear for everything
+    that reads it, with the gated units made in its epilogue, and one for both outputs, [o | down] on the columns
+    [mixer | units]. mlp: None or a dict with gate, up [F, D], down [D, F]; limit: its clamp."""
+
+    def __init__(self, mixer, mlp, limit, dtype, device):
+        self.mixer, self.limit = mixer, float(limit) if mlp is not None else 0.0
+        mat = lambda t: t.to(device, dtype)
+        rows, bias, cols = [mixer.rows], mixer.rows_bias, [mixer.o]
+        self.act_from, self.units = mixer.rows.shape[0], 0
+        if mlp is not None:
+            gate, up = pad_matrix(mat(mlp["gate"])), pad_matrix(mat(mlp["up"]))
+            self.units = gate.shape[0]
+            rows.append(torch.stack([gate, up], 1).reshape(2 * self.units, -1))
+            cols.append(pad_matrix(mat(mlp["down"]), 1, 8))
+            if bias is not None:
+                bias = torch.nn.functional.pad(bias, (0, 2 * self.units))
+        self.w_in, self.bias_in = torch.cat(rows, 0).contiguous(), bias
+        self.w_out = pad_matrix(torch.cat(cols, 1), 8, 1)
+        mixer.rows = None  # part of w_in now
+        self.mixer_cols = mixer.o.shape[1]
+        self.padded = self.mixer_cols != mixer.heads * mixer.vdim
+        mixer.o = None
+
+    def forward(self, s, lc, cache, step, add, norm):
+        T, dev = step.B * step.S, s.h.device
+        sc = _timers.scope
+        cat = (torch.zeros if self.padded else torch.empty)((T, self.mixer_cols + self.units), dtype=s.h.dtype, device=dev)
+        with sc("parallel_in", 0, 0):
+            if self.units:
+                proj = linear_glu(s.h, self.w_in, self.bias_in, self.act_from, self.limit, cat[:, self.mixer_cols:])
+            else:
+                proj = linear(s.h, self.w_in, self.bias_in)
+        with sc("mixer", 0, 0):
+            self.mixer.forward(proj, cat, lc, cache, step)
+        with sc("parallel_out", 0, 0):
+            x, h = linear_residual(cat, self.w_out, s.x, add, norm)
+        return NormedStream(step.B, step.S, x, h)
+
+
+class ParallelDecoderLayer:
+    """x <- x + (mixer(h) + mlp(h)), h the norm of x. One run of a block: several runs may share a block (a looped stack of
+    layers), each with the cache `idx` of its own. add, norm: the vector that comes onto the stream behind this run (or None)
+    and the norm (alpha, w, b) of what reads it next."""
+
+    def __init__(self, idx, block, add, norm):
+        self.idx, self.block, self.add, self.norm = idx, block, add, norm
+
+    def reserve(self, cache, B, tokens, device):
+        self.block.mixer.reserve(cache.hybrid_layer(self.idx), B, tokens, device)
+
+    def forward(self, inp, cache, use_cache=True, dev_len=None):
+        """inp = [NormedStream, start int32 [B] or None, ...]: the interface of the other decoder layers."""
+        s, start = inp[0], inp[1]
+        lc = cache.hybrid_layer(self.idx)
+        s = self.block.forward(s, lc, cache, Step(s.B, s.S, lc.offset, start, dev_len), self.add, self.norm)
+        if dev_len is None:
+            lc.offset += s.S
         return [s]

@@ -128,16 +128,17 @@ class LayerCache:
 
 
 class HybridLayerCache:
-    """What a layer of a hybrid decoder keeps per sequence: latent rows in 32-token pages (latent attention) and named
-    32-bit state tensors [B, ...] that every token updates in place (convolution inputs, the matrix state of a recurrence).
+    """What a layer of a hybrid decoder keeps per sequence: rows in 32-token pages (latents, or keys and values side by side)
+    and named 32-bit state tensors [B, ...] that every token updates in place (convolution inputs, the matrix state of a
+    recurrence).
 
-    Pages are [B, 32, R] slabs reached through a device array of addresses, as in LayerCache. With a sliding window only
-    the last `window` tokens are ever read: the page table stops growing at the number of pages a window can touch, and
+    Pages are [B, 32, R] or [B, G, 32, R] slabs reached through a device array of addresses, as in LayerCache. With a sliding
+    window, or chunks of `window` tokens, only the last `window` tokens are ever read: the page table stops growing at the number of pages a window can touch, and
     token t then lives in page (t // 32) mod pages, i.e. old pages are used again. While the table still grows no page index
     has wrapped, so growth moves nothing."""
 
     def __init__(self):
-        self.arenas = []     # tensors [pages, B, 32, R]
+        self.arenas = []     # tensors [pages, B, (G,) 32, R]
         self.ptrs = None     # int64 [pages]
         self.window = 0      # tokens ever looked back at, 0: all
         self.states = {}
@@ -161,9 +162,12 @@ class HybridLayerCache:
         return self.arenas[0].shape[1] if self.arenas else None
 
     def ensure_latent(self, B, R, tokens, window, dtype, device):
-        """Pages for the tokens up to index offset + tokens - 1."""
-        if self.arenas and tuple(self.arenas[0].shape[1:]) != (B, S2, R):
-            raise _lib.TpxError("latent cache shape changed between calls")
+        self.ensure_pages((B, S2, R), tokens, window, dtype, device)
+
+    def ensure_pages(self, slab, tokens, window, dtype, device):
+        """Pages of shape `slab` for the tokens up to index offset + tokens - 1."""
+        if self.arenas and tuple(self.arenas[0].shape[1:]) != tuple(slab):
+            raise _lib.TpxError("cache shape changed between calls")
         self.window = window
         need = (self.offset + tokens + S2 - 1) // S2
         if need > self.pages():
@@ -171,7 +175,7 @@ class HybridLayerCache:
         if window:
             need = min(need, self.window_pages())
         if need > self.pages():
-            self.arenas.append(torch.zeros((need - self.pages(), B, S2, R), dtype=dtype, device=device))
+            self.arenas.append(torch.zeros((need - self.pages(),) + tuple(slab), dtype=dtype, device=device))
             self._rebuild_table()
 
     def _rebuild_table(self):
@@ -195,7 +199,7 @@ class HybridLayerCache:
     def reserve(self, steps):
         if self.arenas:
             a = self.arenas[0]
-            self.ensure_latent(a.shape[1], a.shape[3], steps, self.window, a.dtype, a.device)
+            self.ensure_pages(a.shape[1:], steps, self.window, a.dtype, a.device)
 
     def fits(self, batch, need):
         return self.batch() == batch and self.capacity() >= need

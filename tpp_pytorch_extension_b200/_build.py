@@ -23,7 +23,8 @@ NVCC_FLAGS = [
 
 
 # sources of models that do not need the whole library (names without the tpx_ prefix)
-COMPONENTS = {"Dofivik": ("api", "linear_bf16", "linear_f32", "postnorm", "latent", "latent_tc", "latent_dec", "delta")}
+COMPONENTS = {"Dofivik": ("api", "linear_bf16", "linear_f32", "postnorm", "latent", "latent_tc", "latent_dec", "delta"),
+              "Vedizen": ("api", "linear_bf16", "linear_f32", "postnorm", "dyt", "gla", "diff", "diff_tc", "diff_dec")}
 
 
 def sources():

@@ -82,6 +82,12 @@ _SIGS = {
     "tpx_latent_prefill": (c_int, [c_vp, c_vp]),
     "tpx_latent_tc_status": (c_int, [c_vp, ctypes.POINTER(ctypes.c_uint)]),
     "tpx_delta_rule": (c_int, [c_vp, c_vp]),
+    "tpx_dyt": (c_int, [c_vp, c_vp]),
+    "tpx_gla_token_serves": (c_int, [c_i64] * 2),
+    "tpx_gla": (c_int, [c_vp, c_vp]),
+    "tpx_diff_prefill_serves": (c_int, [c_i64, c_i64, c_f32]),
+    "tpx_diff_attn": (c_int, [c_vp, c_vp]),
+    "tpx_diff_status": (c_int, [c_vp, ctypes.POINTER(ctypes.c_uint)]),
     "tpx_qlinear": (c_int, [c_int, c_vp, c_vp, c_vp, c_vp, c_i64, c_vp, c_i64, c_i64, c_i64, c_vp, c_int, c_vp, c_vp,
                             c_f32, c_vp, c_vp, c_sz, c_vp]),
 }
@@ -140,7 +146,8 @@ def _struct(name, **groups):
     return type(name, (ctypes.Structure,), {"_fields_": [(n, types[g[0]]) for g, names in groups.items() for n in names.split()]})
 
 
-LinearStruct = _struct("LinearStruct", p="w x bias act_params y", l="M N K ldw ldx ldy", i="f32 out_f32 act act_from", p2="scratch", z="scratch_bytes")
+LinearStruct = _struct("LinearStruct", p="w x bias act_params y", l="M N K ldw ldx ldy", i="f32 out_f32 act act_from", p2="scratch", z="scratch_bytes",
+                       p3="z res add norm_w norm_b x_out h", l2="ldz ldr ldh", f="limit norm_alpha")
 PostnormConvStruct = _struct("PostnormConvStruct", p="ids embed x y w conv state start dev_len x_out h", l="B S D ldh past", f="alpha eps", i="taps f32")
 PostnormFinalStruct = _struct("PostnormFinalStruct", p="x y w w_final rows out", l="n D ldo", f="alpha eps", i="f32")
 LatentPrepStruct = _struct("LatentPrepStruct", p="proj q_norm kv_norm freq start dev_len cq cos_sin gate lat pages",
@@ -151,6 +158,12 @@ LatentValueStruct = _struct("LatentValueStruct", p="ol gate w_uv out", l="T head
 LatentPrefillStruct = _struct("LatentPrefillStruct", p="q kv lat cos_sin gate start out",
                               l="B S L past heads dim rot_dim vdim krp R ldq ldkv ldo window", f="scale")
 DeltaRuleStruct = _struct("DeltaRuleStruct", p="proj wraw a_bias norm_w start dev_len state raw out", l="B S past ldp ldo heads dim", f="eps", i="f32")
+
+DytStruct = _struct("DytStruct", p="ids embed x add w b x_out h", l="n D ldh", f="scale alpha", i="f32")
+GlaStruct = _struct("GlaStruct", p="proj zraw a2 a2_bias norm_w start dev_len state raw out",
+                    l="B S past ldp ldo lda2 rank heads dim vdim q_col k_col v_col g_col a1_col", f="tau eps", i="f32")
+DiffAttnStruct = _struct("DiffAttnStruct", p="proj pages live start dev_len out",
+                         l="B S L past npages ldp ldo heads kv_heads dim vdim R chunk q_col k_col v_col", f="scale softcap lam mult eps", i="f32")
 
 
 def check(rc):
@@ -211,7 +224,7 @@ def assert_no_kernel_error(sync=True):
         code = inst.error_code()
         if code:
             raise TpxError(f"the peer-memory all-reduce gave up waiting for rank {code - 1}")
-    for name in ("tpx_attention_tc_status", "tpx_latent_tc_status", "tpx_latent_decode_status"):
+    for name in ("tpx_attention_tc_status", "tpx_latent_tc_status", "tpx_latent_decode_status", "tpx_diff_status"):
         if _lib is not None and hasattr(_lib, name) and torch.cuda.is_available():
             st = ctypes.c_uint(0)
             check(getattr(_lib, name)(stream(), ctypes.byref(st)))

@@ -46,6 +46,12 @@ __device__ __forceinline__ float hy_act(float v, int act, float a0, float a1) {
   }
 }
 
+// one unit of the clamped gated feed-forward
+__device__ __forceinline__ float hy_clamped_glu(float g, float u, float limit) {
+  g = fminf(g, limit);
+  return g * hy_sigmoid(1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+}
+
 // bf16 decoding of latent attention (tpx_latent_dec.cu)
 bool latent_absorb_mma_serves(const TpxLatentAbsorb& a);
 int latent_absorb_mma(const TpxLatentAbsorb& a, cudaStream_t st);
@@ -56,5 +62,11 @@ int latent_decode(const TpxLatentAttn& a, cudaStream_t st);
 
 // the bf16 operands of tpx_linear on the tcgen05 kernel (tpx_linear_bf16.cu)
 int linear_tc_ex(const TpxLinear& a, cudaStream_t st);
+
+// chunked differential attention in bf16: several tokens (tpx_diff_tc.cu), one token, append included (tpx_diff_dec.cu)
+bool diff_prefill_serves(int64_t dim, int64_t vdim, float softcap);
+int diff_prefill(const TpxDiffAttn& a, cudaStream_t st);
+bool diff_decode_serves(const TpxDiffAttn& a);
+int diff_decode(const TpxDiffAttn& a, cudaStream_t st);
 
 }  // namespace tpx

@@ -25,12 +25,19 @@
 
 namespace tpx {
 
-// Epilogue of tpx_linear: fp32 bias, row stride, fp32 or bf16 result, activation from a column on.
+// Epilogue of tpx_linear: fp32 bias, row stride, fp32 or bf16 result, activation from a column on; gated units from pairs of
+// columns; or the residual sum with the norm of its next reader.
 struct BfEx {
   const float *bias, *ap;
   void* y;
   long long ldy;
   int on, out_f32, act, act_from;
+  uint16_t* z;
+  const float *res, *add, *nw, *nb;
+  float* x_out;
+  uint16_t* h;
+  long long ldz, ldr, ldh;
+  float limit, nalpha;
 };
 
 struct BfParams {
@@ -75,6 +82,24 @@ __device__ __forceinline__ void bf_finish16_ex(const BfEx& e, int M, int tok0, i
   float x[16];
 #pragma unroll
   for (int j = 0; j < 16; j++) x[j] = v[j] + b;
+  if (e.x_out) {
+    const float add = e.add ? e.add[n] : 0.0f, w = e.nw[n], nb = e.nb[n];
+    const float* r = e.res + (long long)tok0 * e.ldr + n;
+    float* xo = e.x_out + (long long)tok0 * e.ldr + n;
+    uint16_t* h = e.h + (long long)tok0 * e.ldh + n;
+    float s[16];
+#pragma unroll
+    for (int j = 0; j < 16; j++) s[j] = j < live ? __ldcs(r + j * e.ldr) : 0.0f;
+#pragma unroll
+    for (int j = 0; j < 16; j++) {
+      s[j] += x[j] + add;
+      if (j < live) xo[j * e.ldr] = s[j];
+    }
+#pragma unroll
+    for (int j = 0; j < 16; j++)
+      if (j < live) h[j * e.ldh] = f32_to_bf16_bits(fmaf(tanhf(e.nalpha * s[j]), w, nb));
+    return;
+  }
   if (e.act && n >= e.act_from) {
     const float a0 = e.ap ? e.ap[0] : 0.0f, a1 = e.ap ? e.ap[1] : 0.0f;
 #pragma unroll
@@ -90,6 +115,21 @@ __device__ __forceinline__ void bf_finish16_ex(const BfEx& e, int M, int tok0, i
 #pragma unroll
     for (int j = 0; j < 16; j++)
       if (j < live) y[j * e.ldy] = f32_to_bf16_bits(x[j]);
+  }
+}
+
+// The same where the features are pairs (g, u) of neighbouring lanes: the lane of g finishes the first eight tokens, the lane
+// of u the others. Called by whole warps; lanes with n < act_from take part in the exchange only.
+__device__ __forceinline__ void bf_finish16_glu(const BfEx& e, int M, int N, int tok0, int n, const float (&v)[16]) {
+  const int live = M - tok0, up = n & 1;
+  const float b = (e.bias && n < N) ? e.bias[n] : 0.0f;
+  uint16_t* z = e.z + (long long)(tok0 + up * 8) * e.ldz + (n - e.act_from) / 2;
+#pragma unroll
+  for (int j = 0; j < 8; j++) {
+    const float lo = v[j] + b, hi = v[j + 8] + b;
+    const float other = __shfl_xor_sync(0xffffffffu, up ? lo : hi, 1);
+    const float r = up ? hy_clamped_glu(other, hi, e.limit) : hy_clamped_glu(lo, other, e.limit);
+    if (n >= e.act_from && n < N && up * 8 + j < live) z[j * e.ldz] = f32_to_bf16_bits(r);
   }
 }
 
@@ -253,7 +293,13 @@ linear_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
       const int tok0 = tm * TOK;
       const bool whole = pc.g0 == 0 && pc.g1 == nstages;
       float* part = whole ? nullptr : p.t.partial + ((size_t)blockIdx.x * 2 + (pc.tile == first_tile ? 0 : 1)) * TOK * 128;
+      const bool pairs = p.ex.on && p.ex.act == TPX_ACT_CLAMPED_GLU && tn * 128 + sub * 32 + 31 >= p.ex.act_from;  // per warp
       auto finish = [&](int c0, const float (&v)[16]) {
+        if (pairs) {
+          if (tok0 + c0 >= p.t.M) return;
+          bf_finish16_glu(p.ex, p.t.M, p.t.N, tok0 + c0, n, v);
+          if (n >= p.ex.act_from) return;
+        }
         if (n < p.t.N && tok0 + c0 < p.t.M) {
           const float v2[16] = {};
           if (p.ex.on) bf_finish16_ex(p.ex, p.t.M, tok0 + c0, n, v);
@@ -400,7 +446,8 @@ int linear_tc_ex(const TpxLinear& a, cudaStream_t st) {
               a.scratch_bytes);
   BfParams p = {};
   p.t.err = reinterpret_cast<unsigned*>(reinterpret_cast<unsigned char*>(a.scratch) + kTcCounterBytes - 4);
-  p.ex = {a.bias, a.act_params, a.y, (long long)a.ldy, 1, a.out_f32, a.act, a.act_from};
+  p.ex = {a.bias, a.act_params, a.y, (long long)a.ldy, 1, a.out_f32, a.act, a.act_from, (uint16_t*)a.z, a.res, a.add, a.norm_w, a.norm_b, a.x_out,
+          (uint16_t*)a.h, (long long)a.ldz, (long long)a.ldr, (long long)a.ldh, a.limit, a.norm_alpha};
   return bf_run(p, a.w, a.x, a.M, a.N, a.K, a.ldw, a.ldx, a.scratch, a.scratch_bytes, st);
 }
 

@@ -22,10 +22,13 @@ from tpp_pytorch_extension_b200._C import _fused_llm_infer as fused_llm_cpp
 from tpp_pytorch_extension_b200.llm import fused_dofivik_infer as FD
 from tpp_pytorch_extension_b200.llm import fused_gptj_infer as FG
 from tpp_pytorch_extension_b200.llm import fused_opt_infer as FO
+from tpp_pytorch_extension_b200.llm import fused_vedizen_infer as FV
 
 MODELS = {"llama2-7b": FL.LLAMA2_7B, "llama3-8b": FL.LLAMA3_8B, "llama2-70b": FL.LLAMA2_70B,
           "opt-6.7b": FO.OPTShape(32, 4096, 32, 16384, 50272), "opt-30b": FO.OPTShape(48, 7168, 56, 28672, 50272),
-          "gptj-6b": FG.GPTJShape(28, 4096, 16, 16384, 50400, 64), "dofivik-8b": FD.DOFIVIK_8B}
+          "gptj-6b": FG.GPTJShape(28, 4096, 16, 16384, 50400, 64), "dofivik-8b": FD.DOFIVIK_8B,
+          "vedizen-8b": FV.VEDIZEN_8B}
+HYBRID = (FD.DofivikShape, FV.VedizenShape)  # families whose weights stay in the activation type
 
 
 def main(argv=None):
@@ -58,7 +61,7 @@ def main(argv=None):
     dtype = getattr(torch, a.dtype)
     if a.layers:
         import dataclasses
-        shape = dataclasses.replace(shape, layers=shape.layers[:a.layers]) if isinstance(shape, FD.DofivikShape) else dataclasses.replace(shape, num_hidden_layers=a.layers)
+        shape = dataclasses.replace(shape, layers=shape.layers[:a.layers]) if isinstance(shape, HYBRID) else dataclasses.replace(shape, num_hidden_layers=a.layers)
     wd = {"bfloat16": "bf16"}.get(a.weight_dtype, a.weight_dtype)
     from tpp_pytorch_extension_b200.llm import llm_common
     if a.load_sharded_model:
@@ -68,10 +71,12 @@ def main(argv=None):
         name = model_registry.architecture_of(a.model_dir)
         if dtype not in model_registry.dtypes_of(name):
             ap.error(f"{name} does not run in {a.dtype}")
-        model = model_registry.load_model(a.model_dir, dtype, "cuda", None if name == "Dofivik" else wd)
+        model = model_registry.load_model(a.model_dir, dtype, "cuda", wd if model_registry.quantizes(name) else None)
         shape, a.model = model.shape, name
     elif isinstance(shape, FD.DofivikShape):
         model = FD.build_random_dofivik(shape, dtype, "cuda")
+    elif isinstance(shape, FV.VedizenShape):
+        model = FV.build_random_vedizen(shape, dtype, "cuda")
     elif isinstance(shape, FO.OPTShape):
         model = FO.build_random_opt(shape, wd, "cuda")
     elif isinstance(shape, FG.GPTJShape):
@@ -104,7 +109,7 @@ def main(argv=None):
     per_tok = (tn - t1) / steps
     if rank == 0:
         print(json.dumps({
-            "model": a.model, "weight_dtype": a.dtype if isinstance(shape, FD.DofivikShape) else a.weight_dtype, "tp": world, "layers": shape.num_hidden_layers,
+            "model": a.model, "weight_dtype": a.dtype if isinstance(shape, HYBRID) else a.weight_dtype, "tp": world, "layers": shape.num_hidden_layers,
             "batch_size": a.batch_size, "input_tokens": a.input_tokens, "max_new_tokens": a.max_new_tokens,
             "graph": not a.no_graph, "first_token_ms": round(t1 * 1e3, 3), "next_token_ms": round(per_tok * 1e3, 4),
             "decode_tokens_per_s": round(a.batch_size / per_tok, 1),

@@ -12,9 +12,8 @@ from dataclasses import dataclass, field
 import torch
 
 from .._C import _hybrid_layers as hybrid
-from . import llm_common
-from .fused_llama_infer import LlamaRunner
-from .llm_common import TppCache, get_size
+from .hybrid_runner import HybridRunner
+from .llm_common import get_size
 
 
 @dataclass
@@ -84,73 +83,20 @@ def make_layer(shape, idx, w, norms, device):
     return hybrid.HybridDecoderLayer(idx, norms, mixer, conv("canon1"), vec("norm1"), mlp, conv("canon2"), vec("norm2"))
 
 
-class DofivikRunner(LlamaRunner):
-    packable = False
-
+class DofivikRunner(HybridRunner):
     def __init__(self, shape, embed, layers, norms, final_w, head_w):
-        super().__init__(shape, embed, layers, final_w, head_w, None)
+        super().__init__(shape, embed, layers, final_w, head_w, norms.dtype)
         self.norms = norms
-        self.layer_outputs = None  # a list: receives the stream [B * S, D] after every layer of the next forward calls
-
-    @property
-    def dtype(self):
-        return self.norms.dtype
 
     def _embed(self, ids, positions):
         return hybrid.Stream(ids.shape[0], ids.shape[1], ids=ids.contiguous(), embed=self.embed)
 
     def _head(self, s):
-        """fp32 logits of the wanted rows: [B, 1, V] (last token), [B, S, V], or [rows, V] with logit_rows."""
         B, S, _ = s.shape
-        dev = s.x.device
-        rows = self.logit_rows
-        if rows is None:
-            rows = torch.arange(B * S, device=dev)
-            if self.only_last_logit:
-                rows = rows[S - 1::S].contiguous()
-        logits = hybrid.linear(self.norms.final(s, self.norm_w, rows), self.lm_head_w, out_f32=True)
-        return logits if self.logit_rows is not None else logits.view(B, -1, logits.shape[-1])
+        return self._logits(self.norms.final(s, self.norm_w, self._wanted_rows(B, S, s.x.device)), B)
 
-    def _pick(self, logits):
-        return hybrid.argmax_rows_f32(logits[:, -1]).unsqueeze(-1)
-
-    def _reserve(self, cpp, batch, tokens, device):
-        for layer in self.layers:
-            layer.reserve(cpp, batch, tokens, device)
-
-    def _decode_mask(self, cpp, mask, past, cap):
-        return cpp.start
-
-    @staticmethod
-    def _padding(attention_mask):
-        """Leading padding per sequence from a keep-mask; a state cannot skip tokens in the middle."""
-        keep = attention_mask.to(torch.int64)
-        start = keep.shape[1] - keep.sum(-1)
-        if not torch.equal(keep, (torch.arange(keep.shape[1], device=keep.device) >= start.unsqueeze(-1)).to(torch.int64)):
-            raise ValueError("sequences must be padded on the left")
-        return start.to(torch.int32).contiguous()
-
-    @torch.no_grad()
-    def forward(self, input_ids, attention_mask=None, position_ids=None, cache=None):
-        """Logits of a call's tokens and the cache behind them. attention_mask [B, S] (1 = token, 0 = left padding) counts
-        at a sequence's first call; positions follow from it."""
-        cache = TppCache() if cache is None else cache
-        cpp = cache.get_cpp()
-        B, S = input_ids.shape
-        if input_ids.numel() and (int(input_ids.min()) < 0 or int(input_ids.max()) >= self.shape.vocab_size):
-            raise ValueError("token id outside the vocabulary")
-        if cpp.get_seq_length() == 0:
-            cpp.start = torch.zeros(B, dtype=torch.int32, device=input_ids.device) if attention_mask is None else self._padding(attention_mask)
-        if cpp.start.shape[0] != B:
-            raise ValueError(f"the cache holds {cpp.start.shape[0]} sequences, the call has {B}")
-        s = self._embed(input_ids, None)
-        for layer in self.layers:
-            s = layer.forward([s, cpp.start], cpp, True)[0]
-            if self.layer_outputs is not None:
-                self.layer_outputs.append(self.norms.enter(s, None, None, cpp.start, None, cpp.get_seq_length() - S)[0])
-        for lc in cpp.layers:
-            lc.live = None
-        return self._head(s), cache
+    def _stream_rows(self, s, layer, cpp, past):
+        return self.norms.enter(s, None, None, cpp.start, None, past)[0]
 
 
 def _from_tensors(shape, tensors, dtype, device):

@@ -5,11 +5,14 @@ import os
 import torch
 
 
-def _dofivik(path, dtype, device, weight_dtype):
-    from . import fused_dofivik_infer as FD
-    if weight_dtype not in (None, "bf16", "bfloat16"):
-        raise ValueError("this model family runs on its bfloat16 (or float32) weights: no quantized weight_dtype")
-    return FD.load_dofivik(path, dtype, device)
+def _plain_weights(module, entry):
+    def load(path, dtype, device, weight_dtype):
+        if weight_dtype not in (None, "bf16", "bfloat16"):
+            raise ValueError("this model family runs on its bfloat16 (or float32) weights: no quantized weight_dtype")
+        import importlib
+        return getattr(importlib.import_module("." + module, __package__), entry)(path, dtype, device)
+    load.quantizes = False
+    return load
 
 
 def _hugging_face(module, entry):
@@ -26,7 +29,8 @@ def _hugging_face(module, entry):
 
 # architecture -> (loader, activation types it runs in)
 ARCHITECTURES = {
-    "Dofivik": (_dofivik, (torch.bfloat16, torch.float32)),
+    "Dofivik": (_plain_weights("fused_dofivik_infer", "load_dofivik"), (torch.bfloat16, torch.float32)),
+    "Vedizen": (_plain_weights("fused_vedizen_infer", "load_vedizen"), (torch.bfloat16, torch.float32)),
     "LlamaForCausalLM": (_hugging_face("fused_llama_infer", "OptimizeModelForLlama"), (torch.bfloat16,)),
     "Qwen2ForCausalLM": (_hugging_face("fused_llama_infer", "OptimizeModelForQwen2"), (torch.bfloat16,)),
     "OPTForCausalLM": (_hugging_face("fused_opt_infer", "OptimizeModelForOPT"), (torch.bfloat16,)),
@@ -45,6 +49,11 @@ def architecture_of(path):
 
 def dtypes_of(name):
     return ARCHITECTURES[name][1]
+
+
+def quantizes(name):
+    """Whether the family takes a quantized weight_dtype."""
+    return getattr(ARCHITECTURES[name][0], "quantizes", True)
 
 
 def load_model(path, dtype=torch.bfloat16, device="cuda", weight_dtype=None):
