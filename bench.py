@@ -438,18 +438,111 @@ def hybrid_ops(dev, batch, context, heads=32, width=4096, window=2048):
     return out
 
 
-def hybrid_legs(dev, steps):
-    """Prefill and decode throughput of the hybrid decoder (bf16 random weights) beside a bf16 Llama of the same depth,
-    width, feed-forward, heads and vocabulary."""
+def vedizen_ops(dev, batch, context, heads=32, width=4096, ff=14336, chunk=2048):
+    """The Vedizen decoder's own kernels at one layer's sizes beside the like kernels of the Llama and the Dofivik model (as
+    hybrid_ops): gated linear attention beside the delta rule, differential attention beside the Llama's, the two fused linears
+    beside plain ones of the same shape."""
+    import torch
+    from tpp_pytorch_extension_b200 import _lib
+    from tpp_pytorch_extension_b200._C import _hybrid_layers as HL
+    from tpp_pytorch_extension_b200._C import _tpp_attn as A
+    pk = peaks()
+    bf = lambda *s: torch.randn(*s, device=dev).to(torch.bfloat16)
+    T, out = batch * context, {}
+
+    def put(name, us, bytes_=0, tensor=0, fp32=0):
+        roof = max(bytes_ / (pk["hbm_gbs"] * 1e9), tensor / (pk["bf16_tflops"] * 1e12), fp32 / 72.6e12) * 1e6
+        out[name] = {"us": round(us, 1), "roofline_us": round(roof, 1), "frac": round(roof / us, 3)}
+
+    # linears: into gated units and mixer columns, and from both into the residual stream
+    d, e = 64, 128
+    H = heads
+    n_mix = 2 * H * d + 2 * H * e + 16
+    for name, rows in (("prefill", T), ("decode", batch)):
+        h, res = bf(rows, width), torch.randn(rows, width, device=dev)
+        w_in, w_out = bf(n_mix + 2 * ff, width), bf(width, H * e + ff)
+        cat, norm = bf(rows, H * e + ff), (0.5, torch.ones(width, device=dev), torch.zeros(width, device=dev))
+        n = 10 if rows == T else 40
+        put(f"linear_in_{name}", _time_us(lambda: HL.linear_glu(h, w_in, None, n_mix, 7.0, cat[:, H * e:]), n),
+            2 * (w_in.numel() + h.numel() + rows * (n_mix + ff)), tensor=2 * rows * w_in.numel())
+        put(f"linear_in_{name}_plain", _time_us(lambda: HL.linear(h, w_in), n), 2 * (w_in.numel() + h.numel() + rows * w_in.shape[0]),
+            tensor=2 * rows * w_in.numel())
+        put(f"linear_out_{name}", _time_us(lambda: HL.linear_residual(cat, w_out, res, None, norm), n),
+            2 * (w_out.numel() + cat.numel()) + rows * width * 10, tensor=2 * rows * w_out.numel())
+        put(f"linear_out_{name}_plain", _time_us(lambda: HL.linear(cat, w_out, out_f32=True), n), 2 * (w_out.numel() + cat.numel()) + rows * width * 4,
+            tensor=2 * rows * w_out.numel())
+        del h, res, w_in, w_out, cat
+    # gated linear attention
+    one = torch.ones(e, device=dev)
+    a2, a2b = bf(H * d, 16), torch.ones(H * d, device=dev)
+    for name, B, S in (("prefill", batch, context), ("prefill_batch1", 1, 2 * context), ("decode", batch, 1), ("decode_batch64", 64, 1)):
+        TT = B * S
+        proj, zraw = bf(TT, n_mix), torch.randn(TT, H * d, device=dev)
+        state, o, raw = torch.zeros(B, H, d, e, device=dev), bf(TT, H * e), torch.empty(TT, H * e, device=dev)
+
+        def gla():
+            HL._call("tpx_gla", _lib.GlaStruct(
+                proj=proj.data_ptr(), zraw=zraw.data_ptr() if S > 1 else None, a2=a2.data_ptr(), a2_bias=a2b.data_ptr(), norm_w=one.data_ptr(),
+                state=state.data_ptr(), raw=raw.data_ptr(), out=o.data_ptr(), B=B, S=S, past=0, ldp=n_mix, ldo=H * e, lda2=16, rank=16, heads=H, dim=d,
+                vdim=e, q_col=0, k_col=H * d, v_col=2 * H * d, g_col=2 * H * d + H * e, a1_col=n_mix - 16, tau=16.0, eps=1e-5, f32=0))
+        put(f"gla_{name}", _time_us(gla, 10 if S > 1 else 40), TT * H * (d * 8 + e * 6) + B * H * d * e * 8, fp32=4 * TT * H * d * e)
+        del proj, zraw, state, o, raw
+    TT, dd = T, 64
+    Hd = width // dd
+    proj, wraw, o = bf(TT, 5 * width + 64), torch.randn(TT, width, device=dev), bf(TT, width)
+    onew, zero, state = torch.ones(width, device=dev), torch.zeros(width, device=dev), torch.zeros(batch, Hd, dd, dd, device=dev)
+    for name, S in (("prefill", context), ("decode", 1)):
+        put(f"delta_{name}", _time_us(lambda: HL._call("tpx_delta_rule", _lib.DeltaRuleStruct(
+            proj=proj.data_ptr(), wraw=wraw.data_ptr(), a_bias=zero.data_ptr(), norm_w=onew.data_ptr(), state=state.data_ptr(), raw=wraw.data_ptr(),
+            out=o.data_ptr(), B=batch, S=S, past=0, ldp=proj.shape[1], ldo=width, heads=Hd, dim=dd, eps=1e-6, f32=0)), 10 if S > 1 else 40),
+            batch * S * width * 16 + batch * Hd * dd * dd * 8, fp32=2 * batch * S * width * dd * 4)
+    del proj, wraw, o, state
+    # attention
+    pairs = sum(i % chunk + 1 for i in range(context))
+    R = 2 * d + e + 8
+    for G in (H, H // 4):
+        q, k, v = 0, 2 * H * d, 2 * H * d + 2 * G * d
+        ldp = v + G * e
+
+        def diff(B, S, past, P, pages, ptrs, proj, o):
+            HL._call("tpx_diff_attn", _lib.DiffAttnStruct(
+                proj=proj.data_ptr(), pages=ptrs.data_ptr(), out=o.data_ptr(), B=B, S=S, L=S, past=past, npages=P, ldp=ldp, ldo=H * e, heads=H, kv_heads=G,
+                dim=d, vdim=e, R=R, chunk=chunk, q_col=q, k_col=k, v_col=v, scale=d ** -0.5, softcap=30.0, lam=0.5, mult=0.5, eps=1e-5, f32=0))
+        P = (chunk + 30) // 32 + 1
+        for name, B, S, past in (("prefill", batch, context, 0), ("decode", batch, 1, 2 * chunk - 1), ("decode_batch64", 64, 1, 2 * chunk - 1)):
+            pages = bf(P, B, G, 32, R)
+            ptrs = torch.tensor([pages.data_ptr() + i * pages.stride(0) * 2 for i in range(P)], device=dev)
+            proj, o = bf(B * S, ldp), bf(B * S, H * e)
+            put(f"diff_attn_{name}_kv{G}", _time_us(lambda: diff(B, S, past, P, pages, ptrs, proj, o), 10 if S > 1 else 40),
+                2 * B * S * (ldp + H * e + G * R) if S > 1 else 2 * B * chunk * G * (2 * d + e), tensor=2 * B * H * (pairs if S > 1 else chunk) * 2 * (d + e))
+            del pages, proj, o
+        del ptrs
+    S1, hd = (context + 31) // 32, 128
+    for G in (H, H // 4):
+        k1, v1, q1 = bf(S1, batch, G, 32, hd), bf(S1, batch, G, 32, hd), bf(batch, G, context, H // G, hd)
+        put(f"llama_attn_prefill_kv{G}", _time_us(lambda: A.attention(q1, k1, v1, None, context)), 2 * (2 * k1.numel() + 2 * q1.numel()),
+            tensor=4 * batch * H * hd * context * (context + 1) // 2)
+        q1 = bf(batch, G, 1, H // G, hd)
+        put(f"llama_attn_decode_kv{G}", _time_us(lambda: A.attention(q1, k1, v1, None, context), 40), 2 * 2 * batch * G * context * hd)
+        del k1, v1, q1
+    return out
+
+
+def hybrid_legs(dev, steps, ops, names):
+    """Prefill and decode throughput of the named decoders (bf16 random weights) at the same depth, width, feed-forward, heads
+    and vocabulary."""
     import torch
     from tpp_pytorch_extension_b200.llm import fused_dofivik_infer as FD
     from tpp_pytorch_extension_b200.llm import fused_llama_infer as FL
-    out = {"ops": hybrid_ops(dev, 16, 2048)}
+    from tpp_pytorch_extension_b200.llm import fused_vedizen_infer as FV
+    out = {"ops": ops(dev, 16, 2048)}
     for layers, width, heads, ff, cells in ((8, 4096, 32, 14336, ((16, 2048), (1, 4096))), (16, 2048, 16, 8192, ((16, 1024), (1, 2048)))):
-        for name in ("dofivik", "llama"):
+        for name in names:
             torch.cuda.empty_cache()
             if name == "dofivik":
                 runner = FD.build_random_dofivik(FD.hybrid_shape(layers, width, heads, ff, 32000), device=dev)
+            elif name == "vedizen":
+                runner = FV.build_random_vedizen(FV.vedizen_stack(layers, width, heads, ff, 32000), device=dev)
             else:
                 runner = FL.build_random_llama(FL.LlamaShape(layers, width, heads, heads, ff, 32000, max_position_embeddings=8192), "bf16", dev)
             for batch, context in cells:
@@ -747,7 +840,9 @@ def run_ours(args):
         legs["config5_llama2_70b_mxfp4_tp"] = model_decode_leg("Llama-2-70B shape, MXFP4, tensor parallel", shape, 64, 4096, args.model_steps, dev,
                                                                world, rank, False)
     if "hybrid" in want and world == 1:
-        legs["hybrid_decoder_bf16"] = hybrid_legs(dev, args.model_steps)
+        legs["hybrid_decoder_bf16"] = hybrid_legs(dev, args.model_steps, hybrid_ops, ("dofivik", "llama"))
+    if "vedizen" in want and world == 1:
+        legs["vedizen_decoder_bf16"] = hybrid_legs(dev, args.model_steps, vedizen_ops, ("vedizen", "dofivik", "llama"))
     if rank == 0:
         line["decode_models"] = legs
         print(json.dumps(line))
@@ -763,7 +858,7 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--ms", default="", help="comma-separated subset of the token counts to run (for profiler captures)")
     ap.add_argument("--legs", default="cfg3,cfg4,cfg5", help="model-level decode legs to run after the op sweep: cfg3 (Llama-2-7B shape, int8, one GPU), cfg4 (Llama-3-8B shape, one GPU), "
-                    "cfg5 (Llama-2-70B shape, tensor parallel over --gpus ranks), hybrid (not in the default: the hybrid decoder beside a bf16 Llama of equal size, one GPU); empty for none")
+                    "cfg5 (Llama-2-70B shape, tensor parallel over --gpus ranks), hybrid, vedizen (not in the default: the Dofivik or the Vedizen decoder beside bf16 models of equal size, one GPU); empty for none")
     ap.add_argument("--model-steps", type=int, default=48, help="decode steps timed in each model-level leg")
     ap.add_argument("--cfg5-layers", type=int, default=0, help="decoder layers of the 70B-shape leg (0 = all 80)")
     ap.add_argument("--min-seconds", type=float, default=1.0, help="repeat the K timed steps until this much device time was measured")

@@ -139,7 +139,7 @@ def random_model(cfg, seed=0, gain=1.0, rank=5):
 
     def put(name, *shape, std=None, mean=0.0):
         std = std if std is not None else shape[-1] ** -0.5
-        w[name] = (torch.randn(*shape, generator=g, dtype=torch.float64) * std + mean).to(torch.bfloat16).to(torch.float64)
+        w[name] = (torch.randn(shape, generator=g, dtype=torch.float64) * std + mean).to(torch.bfloat16).to(torch.float64)
 
     def norm(name):
         put(name, D, std=0.2, mean=1.0)

@@ -33,7 +33,7 @@ template <int DS, int VS>
 struct DtCfg {
   static constexpr int SLAB = 128 * 128;  // 128 rows x 64 bf16
   static constexpr int Q_BYTES = 2 * DS * SLAB, SLOT = (DS > VS ? DS : VS) * SLAB;
-  static constexpr int FIT = (224 * 1024 - Q_BYTES) / SLOT, SLOTS = FIT > 6 ? 6 : FIT;
+  static constexpr int FIT = (221 * 1024 - Q_BYTES) / SLOT, SLOTS = FIT > 6 ? 6 : FIT;
   static constexpr size_t SMEM = Q_BYTES + (size_t)SLOTS * SLOT + 1024;
   static constexpr uint32_t COL_S = 0, COL_O = 256;
   static_assert(SLOTS >= 4, "tiles in flight");
