@@ -33,6 +33,30 @@ __global__ void __launch_bounds__(128) diff_append_kernel(TpxDiffAttn p) {
   }
 }
 
+// The same in 16-byte units, for bf16 head sizes that are multiples of 8: a thread per unit of a row.
+__global__ void __launch_bounds__(256) diff_append_v8_kernel(TpxDiffAttn p, int64_t row0) {
+  pdl_trigger();
+  pdl_wait();
+  const int ur = (int)p.R / 8, d8 = (int)p.dim / 8, dp8 = (int)((p.dim + 15) / 16 * 2), v8 = (int)p.vdim / 8, G = (int)p.kv_heads;
+  const int64_t idx = (int64_t)blockIdx.x * 256 + threadIdx.x;
+  const int64_t rg = idx / ur;  // (sequence, token from row0 on, head)
+  const int u = (int)(idx % ur), g = (int)(rg % G);
+  const int64_t n = p.S - row0, bs = rg / G, b = bs / n, s = row0 + bs % n;
+  if (b >= p.B) return;
+  const int64_t past = p.dev_len ? *p.dev_len : p.past, t = past + s;
+  const uint4* pr = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.proj) + (b * p.S + s) * p.ldp);
+  const int m = u / dp8, c = u % dp8;
+  uint4 v = make_uint4(0, 0, 0, 0);
+  if (m < 2) {
+    if (c < d8) v = pr[p.k_col / 8 + (g * 2 + m) * d8 + c];
+  } else if (u - 2 * dp8 < v8) {
+    v = pr[p.v_col / 8 + g * v8 + u - 2 * dp8];
+  }
+  if (t / 32 > (past + p.S - 1) / 32 - p.npages)
+    reinterpret_cast<uint4*>(p.pages[(t / 32) % p.npages])[((b * G + g) * 32 + t % 32) * ur + u] = v;
+  if (p.live) reinterpret_cast<uint4*>(p.live)[((b * p.L + (p.L - p.S) + s) * G + g) * ur + u] = v;
+}
+
 // the cached tokens past - n .. past - 1 into rows 0 .. n - 1 of live; runs before the append, which may use their pages again
 template <typename T>
 __global__ void __launch_bounds__(128) diff_gather_kernel(TpxDiffAttn p) {
@@ -166,8 +190,18 @@ extern "C" int tpx_diff_attn(const TpxDiffAttn* a, void* stream) {
       TPX_CUDA_OK(launch_pdl(k, dim3((unsigned)(a->L - a->S), (unsigned)a->kv_heads, (unsigned)a->B), dim3(128), 0, st, *a));
     }
   }
-  void (*k)(TpxDiffAttn) = a->f32 ? diff_append_kernel<float> : diff_append_kernel<__nv_bfloat16>;
-  TPX_CUDA_OK(launch_pdl(k, dim3((unsigned)(a->B * a->S), (unsigned)a->kv_heads), dim3(128), 0, st, *a));
+  if (!a->f32 && a->dim % 8 == 0 && a->vdim % 8 == 0 && a->ldp % 8 == 0 && a->k_col % 8 == 0 && a->v_col % 8 == 0 && (((uintptr_t)a->proj | (uintptr_t)a->live) & 15) == 0) {
+    // tokens whose pages the call's later tokens use again need no rows, unless they go to `live`
+    int64_t row0 = a->live || a->dev_len ? 0 : (((a->past + a->S - 1) / 32 - a->npages + 1) * 32 - a->past);
+    if (row0 < 0) row0 = 0;
+    const int64_t units = a->B * (a->S - row0) * a->kv_heads * (a->R / 8);
+    TPX_REQUIRE(units < (1ll << 38), TPX_ERR_ARG, "diff_attn: shape too large");
+    TPX_CUDA_OK(launch_pdl(diff_append_v8_kernel, dim3((unsigned)((units + 255) / 256)), dim3(256), 0, st, *a, row0));
+  } else {
+    TPX_REQUIRE(a->kv_heads <= 65535, TPX_ERR_UNSUPPORTED, "diff_attn: too many heads");
+    void (*k)(TpxDiffAttn) = a->f32 ? diff_append_kernel<float> : diff_append_kernel<__nv_bfloat16>;
+    TPX_CUDA_OK(launch_pdl(k, dim3((unsigned)(a->B * a->S), (unsigned)a->kv_heads), dim3(128), 0, st, *a));
+  }
   if (a->S > 1 && !a->f32 && diff_prefill_serves(a->dim, a->vdim, a->softcap)) return diff_prefill(*a, st);
   TpxDiffAttn b = *a;
   if (a->S == 1) b.live = nullptr;

@@ -207,6 +207,19 @@ __global__ void __launch_bounds__(kGlaTokThreads) gla_token_kernel(TpxGla p) {
 }
 
 // ---------------------------------------------------------------- bf16, several tokens
+// the same on the special-function unit; what counts of the logarithm is its absolute error, below 4e-7
+__device__ __forceinline__ float gl_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float gl_decay(float z, float inv_tau) {
+  const float y = z * -1.4426950408889634f;
+  float lg;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(lg) : "f"(1.0f + gl_ex2(-fabsf(y))));
+  return gl_ex2((fmaxf(y, 0.0f) + lg) * -inv_tau);
+}
+__device__ __forceinline__ float gl_silu(float g) { return __fdividef(g, 1.0f + __expf(-g)); }
 __device__ __forceinline__ float2 gl_fma2(float2 a, float2 b, float2 c) {
   unsigned long long r;
   asm("fma.rn.f32x2 %0, %1, %2, %3;"
@@ -246,6 +259,35 @@ __device__ __forceinline__ void gl_ld_bf16(const uint16_t* p, float (&v)[N]) {
   }
 }
 
+template <int N>
+__device__ __forceinline__ void gl_ld_f32(const float* p, float (&v)[N]) {
+  if constexpr (N % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+      const float4 u = *reinterpret_cast<const float4*>(p + i);
+      v[i] = u.x; v[i + 1] = u.y; v[i + 2] = u.z; v[i + 3] = u.w;
+    }
+  } else if constexpr (N == 2) {
+    const float2 u = *reinterpret_cast<const float2*>(p);
+    v[0] = u.x; v[1] = u.y;
+  } else {
+    static_assert(N == 1, "vector size");
+    v[0] = *p;
+  }
+}
+template <int N>
+__device__ __forceinline__ void gl_st_f32(float* p, const float (&v)[N]) {
+  if constexpr (N % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+  } else if constexpr (N == 2) {
+    *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+  } else {
+    static_assert(N == 1, "vector size");
+    *p = v[0];
+  }
+}
+
 // DP: key channels (padded), EC: columns of a CTA, LPC lanes per column, CPT columns per thread, TC tokens staged at once;
 // WHOLE: the CTA has all columns of the head and finishes the output
 template <int DP, int EC, int LPC, int CPT, int TC, bool WHOLE>
@@ -256,7 +298,11 @@ struct GfCfg {
   static constexpr size_t SMEM = STAGED * 4 + 2 * RAW;
   static constexpr int M = 4 * CPT / LPC;  // read-outs a lane ends with per block of four tokens
   static_assert(KPT % 4 == 0 && THREADS % 32 == 0 && LPC <= 32 && 4 * CPT >= LPC && (STAGED * 4) % 16 == 0, "whole vectors and warps");
-  static_assert(M <= CPT || M % CPT == 0, "a lane's read-outs");
+  static_assert(M <= CPT, "a lane's read-outs belong to one token");
+  // 16-byte units that a thread copies: rows of DP bf16, DP fp32, EC bf16; a thread keeps its place in the row
+  static constexpr int UD = DP / 8, UZ = DP / 4, UE = EC / 8;
+  static_assert(THREADS % UD == 0 && THREADS % UZ == 0 && THREADS % UE == 0, "copies");
+  static constexpr int OW = EC / 32;  // columns per lane in the output norm
 };
 
 template <int THREADS>
@@ -279,36 +325,47 @@ __global__ void __launch_bounds__(GfCfg<DP, EC, LPC, CPT, TC, WHOLE>::THREADS) g
   const int dim = (int)p.dim, vdim = (int)p.vdim, S = (int)p.S, ldp = (int)p.ldp, zd = (int)p.heads * dim;
   const int cols = min(EC, vdim - e0);
   const float scale = 1.0f / sqrtf((float)dim), inv_tau = 1.0f / p.tau;
-  constexpr int CH = DP / 32;
+  constexpr int CW = DP / 32;  // channels per lane where a warp has the whole head
   pdl_wait();
   const int first = gla_first(p, b);
   const int64_t row0 = (int64_t)b * S;
-  const uint16_t* proj = reinterpret_cast<const uint16_t*>(p.proj) + row0 * ldp;
-  const float* zraw = p.zraw + row0 * zd + head * dim;
+  const uint16_t* proj = reinterpret_cast<const uint16_t*>(p.proj) + (row0 + first) * ldp;
+  // this thread's places in the rows it copies
+  const uint16_t* fq = proj + (int64_t)(tid / C::UD) * ldp + p.q_col + head * dim + tid % C::UD * 8;
+  const uint16_t* fv = proj + (int64_t)(tid / C::UE) * ldp + p.v_col + head * vdim + e0 + tid % C::UE * 8;
+  const float* fz = p.zraw + (row0 + first + tid / C::UZ) * zd + head * dim + tid % C::UZ * 4;
+  const int64_t kq = p.k_col - p.q_col, gv = p.g_col - p.v_col;
+  const bool inq = tid % C::UD * 8 < dim, inz = tid % C::UZ * 4 < dim, inv = tid % C::UE * 8 < cols;
 
   auto fetch = [&](int t0, int stage) {  // tokens beyond the call and channels beyond the head read as zero
-    unsigned char* dst = raw + stage * C::RAW;
-    const uint16_t* rq = proj + (int64_t)t0 * ldp + p.q_col + head * dim;
-    const uint16_t* rk = proj + (int64_t)t0 * ldp + p.k_col + head * dim;
-    const uint16_t* rv = proj + (int64_t)t0 * ldp + p.v_col + head * vdim + e0;
+    unsigned char* dst = raw + stage * C::RAW + tid * 16;
     const int n = S - t0;
-    for (int i = tid; i < TC * (DP / 8); i += C::THREADS) {
-      const int t = i / (DP / 8), c = i % (DP / 8) * 8;
-      const bool ok = t < n && c < dim;
-      gl_cp16(dst + C::RQ + i * 16, ok ? rq + (int64_t)t * ldp + c : proj, ok);
-      gl_cp16(dst + C::RK + i * 16, ok ? rk + (int64_t)t * ldp + c : proj, ok);
+#pragma unroll
+    for (int i = 0; i < TC; i += C::THREADS / C::UD) {
+      const bool ok = inq && tid / C::UD + i < n && (C::THREADS / C::UD <= TC || tid / C::UD < TC);
+      const uint16_t* src = ok ? fq + (int64_t)i * ldp : proj;
+      if (C::THREADS / C::UD <= TC || tid / C::UD < TC) {
+        gl_cp16(dst + C::RQ + i * DP * 2, src, ok);
+        gl_cp16(dst + C::RK + i * DP * 2, ok ? src + kq : proj, ok);
+      }
     }
-    for (int i = tid; i < TC * (DP / 4); i += C::THREADS) {
-      const int t = i / (DP / 4), c = i % (DP / 4) * 4;
-      const bool ok = t < n && c < dim;
-      gl_cp16(dst + C::RZ + i * 16, ok ? zraw + (int64_t)(t0 + t) * zd + c : zraw, ok);
+#pragma unroll
+    for (int i = 0; i < TC; i += C::THREADS / C::UZ) {
+      const bool ok = inz && tid / C::UZ + i < n;
+      if (C::THREADS / C::UZ <= TC || tid / C::UZ < TC) gl_cp16(dst + C::RZ + i * DP * 4, ok ? (const void*)(fz + (int64_t)i * zd) : proj, ok);
     }
-    for (int i = tid; i < TC * (EC / 8); i += C::THREADS) {
-      const int t = i / (EC / 8), c = i % (EC / 8) * 8;
-      const bool ok = t < n && c < cols;
-      gl_cp16(dst + C::RV + i * 16, ok ? rv + (int64_t)t * ldp + c : proj, ok);
-      if (WHOLE) gl_cp16(dst + C::RG + i * 16, ok ? rv + (int64_t)t * ldp + (p.g_col - p.v_col) + c : proj, ok);
+#pragma unroll
+    for (int i = 0; i < TC; i += C::THREADS / C::UE) {
+      const bool ok = inv && tid / C::UE + i < n;
+      const uint16_t* src = ok ? fv + (int64_t)i * ldp : proj;
+      if (C::THREADS / C::UE <= TC || tid / C::UE < TC) {
+        gl_cp16(dst + C::RV + i * EC * 2, src, ok);
+        if (WHOLE) gl_cp16(dst + C::RG + i * EC * 2, ok ? src + gv : proj, ok);
+      }
     }
+    fq += (int64_t)TC * ldp;
+    fv += (int64_t)TC * ldp;
+    fz += (int64_t)TC * zd;
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (first < S) fetch(first, 0);
@@ -317,6 +374,10 @@ __global__ void __launch_bounds__(GfCfg<DP, EC, LPC, CPT, TC, WHOLE>::THREADS) g
     for (int i = tid; i < first * vdim; i += C::THREADS) out[(int64_t)(i / vdim) * p.ldo + i % vdim] = 0;
   }
 
+  float nw[WHOLE ? C::OW : 1];
+  if (WHOLE)
+#pragma unroll
+    for (int i = 0; i < C::OW; i++) nw[i] = lane * C::OW + i < vdim ? __ldg(p.norm_w + lane * C::OW + i) : 0.0f;
   float2 s[CPT][KP];  // [column][pair of key channels]
   float* st = p.state + ((int64_t)(b * p.heads + head) * dim) * vdim + e0 + c0;
 #pragma unroll
@@ -344,47 +405,54 @@ __global__ void __launch_bounds__(GfCfg<DP, EC, LPC, CPT, TC, WHOLE>::THREADS) g
     if (t0 + TC < S) fetch(t0 + TC, stage ^ 1);
     const unsigned char* rw = raw + stage * C::RAW;
     const uint16_t* rv = reinterpret_cast<const uint16_t*>(rw + C::RV);
-    // the vectors of a block of four tokens: a warp per block, channels lane, lane + 32, ...
+    // the vectors of a block of four tokens: a warp per block, neighbouring channels per lane
     for (int blk = warp; blk < C::NB; blk += C::NW) {
-      const uint16_t* rq = reinterpret_cast<const uint16_t*>(rw + C::RQ) + blk * 4 * DP;
-      const uint16_t* rk = reinterpret_cast<const uint16_t*>(rw + C::RK) + blk * 4 * DP;
-      const float* rz = reinterpret_cast<const float*>(rw + C::RZ) + blk * 4 * DP;
-      float d[16];
+      const int c = lane * CW;
+      const uint16_t* rq = reinterpret_cast<const uint16_t*>(rw + C::RQ) + blk * 4 * DP + c;
+      const uint16_t* rk = reinterpret_cast<const uint16_t*>(rw + C::RK) + blk * 4 * DP + c;
+      const float* rz = reinterpret_cast<const float*>(rw + C::RZ) + blk * 4 * DP + c;
+      float q[4][CW], k[4][CW], a[4][CW], d[16];
+#pragma unroll
+      for (int t = 0; t < 4; t++) {
+        gl_ld_bf16<CW>(rq + t * DP, q[t]);
+        gl_ld_bf16<CW>(rk + t * DP, k[t]);
+        gl_ld_f32<CW>(rz + t * DP, a[t]);
+#pragma unroll
+        for (int i = 0; i < CW; i++) {
+          q[t][i] *= scale;
+          a[t][i] = blk * 4 + t < n ? gl_decay(a[t][i], inv_tau) : 1.0f;
+        }
+      }
 #pragma unroll
       for (int i = 0; i < 16; i++) d[i] = 0.0f;
 #pragma unroll
-      for (int i = 0; i < CH; i++) {
-        const int c = lane + 32 * i;
-        float q[4], k[4], a[4];
+      for (int t = 0; t < 4; t++)
 #pragma unroll
-        for (int t = 0; t < 4; t++) {
-          q[t] = bf16_bits_to_f32(rq[t * DP + c]) * scale;
-          k[t] = bf16_bits_to_f32(rk[t * DP + c]);
-          a[t] = blk * 4 + t < n ? gla_decay(rz[t * DP + c], inv_tau) : 1.0f;
-        }
-        float f = 1.0f;
-#pragma unroll
-        for (int t = 0; t < 4; t++) {
-          f *= a[t];
-          s_q[(blk * 4 + t) * DP + c] = q[t] * f;
-        }
-        s_a[blk * DP + c] = f;
-        f = 1.0f;
-#pragma unroll
-        for (int t = 3; t >= 0; t--) {
-          s_k[(blk * 4 + t) * DP + c] = k[t] * f;
-          f *= a[t];
-        }
-#pragma unroll
-        for (int t = 0; t < 4; t++) {
-          float x = q[t];
+        for (int i = 0; i < CW; i++) {
+          float x = q[t][i];
 #pragma unroll
           for (int u = t; u >= 0; u--) {
-            d[t * 4 + u] = fmaf(x, k[u], d[t * 4 + u]);
-            x *= a[u];
+            d[t * 4 + u] = fmaf(x, k[u][i], d[t * 4 + u]);
+            x *= a[u][i];
           }
+          q[t][i] = x;  // times the decays from the block's first token to t
         }
+      float f[CW];
+#pragma unroll
+      for (int i = 0; i < CW; i++) f[i] = 1.0f;
+#pragma unroll
+      for (int t = 3; t >= 0; t--)
+#pragma unroll
+        for (int i = 0; i < CW; i++) {
+          k[t][i] *= f[i];
+          f[i] *= a[t][i];
+        }
+#pragma unroll
+      for (int t = 0; t < 4; t++) {
+        gl_st_f32<CW>(s_q + (blk * 4 + t) * DP + c, q[t]);
+        gl_st_f32<CW>(s_k + (blk * 4 + t) * DP + c, k[t]);
       }
+      gl_st_f32<CW>(s_a + blk * DP + c, f);
       // sums over the warp, every step leaving a lane half of its values
 #pragma unroll
       for (int x = 16, m = 8; m > 0; x >>= 1, m >>= 1) {
@@ -462,48 +530,49 @@ __global__ void __launch_bounds__(GfCfg<DP, EC, LPC, CPT, TC, WHOLE>::THREADS) g
             o[i] = mine + __shfl_xor_sync(0xffffffffu, other, x);
           }
       }
-      constexpr int MT = M < CPT ? M : CPT;  // values of one token
+      const int t = l * M / CPT, c = l * M % CPT;
+      const float4 d = *reinterpret_cast<const float4*>(s_d + blk * 16 + t * 4);  // zero for later tokens
+      const float dd[4] = {d.x, d.y, d.z, d.w};
+      float r[M];
 #pragma unroll
-      for (int j = 0; j < M; j += MT) {
-        const int t = (l * M + j) / CPT, c = (l * M + j) % CPT;
-        const float4 d = *reinterpret_cast<const float4*>(s_d + blk * 16 + t * 4);  // zero for later tokens
-        const float dd[4] = {d.x, d.y, d.z, d.w};
+      for (int i = 0; i < M; i++) r[i] = o[i];
 #pragma unroll
-        for (int u = 0; u < 4; u++) {
-          float v[MT];
-          gl_ld_bf16<MT>(rv + (blk * 4 + u) * EC + c0 + c, v);
+      for (int u = 0; u < 4; u++) {
+        float w[M];
+        gl_ld_bf16<M>(rv + (blk * 4 + u) * EC + c0 + c, w);
 #pragma unroll
-          for (int i = 0; i < MT; i++) o[j + i] = fmaf(dd[u], v[i], o[j + i]);
-        }
-        if (WHOLE) {
-#pragma unroll
-          for (int i = 0; i < MT; i++) s_o[(blk * 4 + t) * EC + c0 + c + i] = o[j + i];
-        } else if (blk * 4 + t < n) {
-          float* r = p.raw + ((row0 + t0 + blk * 4 + t) * p.heads + head) * vdim + e0 + c0 + c;
-#pragma unroll
-          for (int i = 0; i < MT; i++)
-            if (c0 + c + i < cols) r[i] = o[j + i];
-        }
+        for (int i = 0; i < M; i++) r[i] = fmaf(dd[u], w[i], r[i]);
       }
+      if (WHOLE) gl_st_f32<M>(s_o + (blk * 4 + t) * EC + c0 + c, r);
+      else if (blk * 4 + t < n && c0 + c < cols) gl_st_f32<M>(p.raw + ((row0 + t0 + blk * 4 + t) * p.heads + head) * vdim + e0 + c0 + c, r);
     }
     if (WHOLE) {
       gl_sync<C::THREADS>();
       // output norm and gate: a warp per token
-      constexpr int OH = (EC + 31) / 32;
       const uint16_t* rg = reinterpret_cast<const uint16_t*>(rw + C::RG);
+      const int c = lane * C::OW;
+      uint16_t* out = reinterpret_cast<uint16_t*>(p.out) + (row0 + t0) * p.ldo + head * vdim + c;
       for (int t = warp; t < n; t += C::NW) {
-        float x[OH], ss = 0.0f;
+        float x[C::OW], g[C::OW], ss = 0.0f;
+        gl_ld_f32<C::OW>(s_o + t * EC + c, x);
+        gl_ld_bf16<C::OW>(rg + t * EC + c, g);
 #pragma unroll
-        for (int i = 0; i < OH; i++) {
-          x[i] = lane + 32 * i < cols ? s_o[t * EC + lane + 32 * i] : 0.0f;
-          ss = fmaf(x[i], x[i], ss);
-        }
-        const float inv = 1.0f / sqrtf(hy_warp_sum(ss) / (float)vdim + p.eps);
-        uint16_t* out = reinterpret_cast<uint16_t*>(p.out) + (row0 + t0 + t) * p.ldo + head * vdim;
+        for (int i = 0; i < C::OW; i++) ss = fmaf(x[i], x[i], ss);
+        if (c >= cols) ss = 0.0f;
+        const float rms = rsqrtf(hy_warp_sum(ss) / (float)vdim + p.eps);
 #pragma unroll
-        for (int i = 0; i < OH; i++) {
-          const int c = lane + 32 * i;
-          if (c < cols) out[c] = f32_to_bf16_bits(x[i] * inv * __ldg(p.norm_w + c) * gla_silu(bf16_bits_to_f32(rg[t * EC + c])));
+        for (int i = 0; i < C::OW; i++) x[i] = x[i] * rms * nw[i] * gl_silu(g[i]);
+        if (c < cols) {
+          uint16_t* dst = out + (int64_t)t * p.ldo;
+          if constexpr (C::OW == 1) {
+            dst[0] = f32_to_bf16_bits(x[0]);
+          } else {
+#pragma unroll
+            for (int i = 0; i < C::OW; i += 2) {
+              const __nv_bfloat162 w = __floats2bfloat162_rn(x[i], x[i + 1]);
+              *reinterpret_cast<__nv_bfloat162*>(dst + i) = w;
+            }
+          }
         }
       }
     }
@@ -551,7 +620,7 @@ static int gla_fast_launch(const TpxGla& p, cudaStream_t st) {
 static bool gla_fast_serves(const TpxGla& a) {
   return !a.f32 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.dim <= 128 && a.ldp % 8 == 0 && a.q_col % 8 == 0 && a.k_col % 8 == 0 && a.v_col % 8 == 0 &&
          a.g_col % 8 == 0 && a.ldp < (1ll << 30) && a.heads * a.dim < (1ll << 30) &&
-         (((uintptr_t)a.proj | (uintptr_t)a.zraw | (uintptr_t)a.state) & 15) == 0;
+         a.ldo % 8 == 0 && (((uintptr_t)a.proj | (uintptr_t)a.zraw | (uintptr_t)a.state | (uintptr_t)a.raw | (uintptr_t)a.out) & 15) == 0;
 }
 
 static int gla_fast(const TpxGla& a, cudaStream_t st) {
@@ -564,8 +633,8 @@ static int gla_fast(const TpxGla& a, cudaStream_t st) {
   }
   if (a.dim <= 64) {
     if (!many) return gla_fast_launch<64, 32, 16, 4, 16, false>(a, st);
-    return a.vdim <= 64 ? gla_fast_launch<64, 64, 4, 8, 8, true>(a, st) : a.vdim <= 128 ? gla_fast_launch<64, 128, 4, 8, 8, true>(a, st)
-                                                                                       : gla_fast_launch<64, 256, 4, 8, 8, true>(a, st);
+    return a.vdim <= 64 ? gla_fast_launch<64, 64, 4, 8, 16, true>(a, st) : a.vdim <= 128 ? gla_fast_launch<64, 128, 4, 8, 16, true>(a, st)
+                                                                                       : gla_fast_launch<64, 256, 4, 8, 16, true>(a, st);
   }
   if (!many) return gla_fast_launch<128, 32, 16, 4, 16, false>(a, st);
   return a.vdim <= 64 ? gla_fast_launch<128, 64, 8, 8, 8, true>(a, st) : a.vdim <= 128 ? gla_fast_launch<128, 128, 8, 8, 8, true>(a, st)

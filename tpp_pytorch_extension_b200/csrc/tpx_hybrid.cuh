@@ -63,6 +63,12 @@ int latent_decode(const TpxLatentAttn& a, cudaStream_t st);
 // the bf16 operands of tpx_linear on the tcgen05 kernel (tpx_linear_bf16.cu)
 int linear_tc_ex(const TpxLinear& a, cudaStream_t st);
 
+// as above for a bf16 result: special-function exponential, approximate quotient
+__device__ __forceinline__ float hy_clamped_glu_fast(float g, float u, float limit) {
+  g = fminf(g, limit);
+  return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+}
+
 // chunked differential attention in bf16: several tokens (tpx_diff_tc.cu), one token, append included (tpx_diff_dec.cu)
 bool diff_prefill_serves(int64_t dim, int64_t vdim, float softcap);
 int diff_prefill(const TpxDiffAttn& a, cudaStream_t st);

@@ -128,7 +128,7 @@ __device__ __forceinline__ void bf_finish16_glu(const BfEx& e, int M, int N, int
   for (int j = 0; j < 8; j++) {
     const float lo = v[j] + b, hi = v[j + 8] + b;
     const float other = __shfl_xor_sync(0xffffffffu, up ? lo : hi, 1);
-    const float r = up ? hy_clamped_glu(other, hi, e.limit) : hy_clamped_glu(lo, other, e.limit);
+    const float r = hy_clamped_glu_fast(up ? other : lo, up ? hi : other, e.limit);
     if (n >= e.act_from && n < N && up * 8 + j < live) z[j * e.ldz] = f32_to_bf16_bits(r);
   }
 }
