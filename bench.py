@@ -472,6 +472,13 @@ def vedizen_ops(dev, batch, context, heads=32, width=4096, ff=14336, chunk=2048)
         put(f"linear_out_{name}_plain", _time_us(lambda: HL.linear(cat, w_out, out_f32=True), n), 2 * (w_out.numel() + cat.numel()) + rows * width * 4,
             tensor=2 * rows * w_out.numel())
         del h, res, w_in, w_out, cat
+    # the start of the stream (embedding, norm) beside the Llama's norm
+    from tpp_pytorch_extension_b200._C import _fused_llm_infer as F
+    table, norm = bf(32000, width), (0.5, torch.ones(width, device=dev), torch.zeros(width, device=dev))
+    ids, xb, gam = torch.randint(0, 32000, (T,), device=dev), bf(T, width), torch.ones(width, device=dev, dtype=torch.bfloat16)
+    put("embed_norm_prefill", _time_us(lambda: HL.dynamic_tanh(norm, torch.bfloat16, ids=ids, embed=table, scale=8.0)), T * width * 8)
+    put("llama_rmsnorm_prefill", _time_us(lambda: F.rms_norm(xb, gam, 1e-5)), T * width * 4)
+    del table, ids, xb
     # gated linear attention
     one = torch.ones(e, device=dev)
     a2, a2b = bf(H * d, 16), torch.ones(H * d, device=dev)
@@ -487,15 +494,14 @@ def vedizen_ops(dev, batch, context, heads=32, width=4096, ff=14336, chunk=2048)
                 vdim=e, q_col=0, k_col=H * d, v_col=2 * H * d, g_col=2 * H * d + H * e, a1_col=n_mix - 16, tau=16.0, eps=1e-5, f32=0))
         put(f"gla_{name}", _time_us(gla, 10 if S > 1 else 40), TT * H * (d * 8 + e * 6) + B * H * d * e * 8, fp32=4 * TT * H * d * e)
         del proj, zraw, state, o, raw
-    TT, dd = T, 64
-    Hd = width // dd
-    proj, wraw, o = bf(TT, 5 * width + 64), torch.randn(TT, width, device=dev), bf(TT, width)
+    dd, Hd = 64, width // 64
+    proj, wraw, o = bf(T, 5 * width + 64), torch.randn(T, width, device=dev), bf(T, width)
     onew, zero, state = torch.ones(width, device=dev), torch.zeros(width, device=dev), torch.zeros(batch, Hd, dd, dd, device=dev)
-    for name, S in (("prefill", context), ("decode", 1)):
+    for name, B, S in (("prefill", batch, context), ("prefill_batch1", 1, 2 * context), ("decode", batch, 1)):
         put(f"delta_{name}", _time_us(lambda: HL._call("tpx_delta_rule", _lib.DeltaRuleStruct(
             proj=proj.data_ptr(), wraw=wraw.data_ptr(), a_bias=zero.data_ptr(), norm_w=onew.data_ptr(), state=state.data_ptr(), raw=wraw.data_ptr(),
-            out=o.data_ptr(), B=batch, S=S, past=0, ldp=proj.shape[1], ldo=width, heads=Hd, dim=dd, eps=1e-6, f32=0)), 10 if S > 1 else 40),
-            batch * S * width * 16 + batch * Hd * dd * dd * 8, fp32=2 * batch * S * width * dd * 4)
+            out=o.data_ptr(), B=B, S=S, past=0, ldp=proj.shape[1], ldo=width, heads=Hd, dim=dd, eps=1e-6, f32=0)), 10 if S > 1 else 40),
+            B * S * width * 16 + B * Hd * dd * dd * 8, fp32=2 * B * S * width * dd * 4)
     del proj, wraw, o, state
     # attention
     pairs = sum(i % chunk + 1 for i in range(context))

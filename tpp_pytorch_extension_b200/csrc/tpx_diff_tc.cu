@@ -108,9 +108,10 @@ __device__ __forceinline__ float2 dt_two(float a) { return make_float2(a, a); }
 // log2 of exp(softcap tanh(s / softcap)) for 32 raw scores; zc: score to s / softcap, uc: score to s log2(e), tc: softcap log2(e).
 // tanh(z) / z on |z| <= 1 is a polynomial in z^2: the interpolant at the Chebyshev nodes of [0, 1], relative error below 1.3e-7.
 __device__ __forceinline__ void dt_capped(uint32_t (&v)[32], float zc, float uc, float tc) {
-  float big = 0.0f;
+  float b4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
-  for (int i = 0; i < 32; i++) big = fmaxf(big, fabsf(__uint_as_float(v[i])));
+  for (int i = 0; i < 32; i += 2) b4[(i >> 1) & 3] = fmaxf(fmaxf(b4[(i >> 1) & 3], fabsf(__uint_as_float(v[i]))), fabsf(__uint_as_float(v[i + 1])));
+  const float big = fmaxf(fmaxf(b4[0], b4[1]), fmaxf(b4[2], b4[3]));
   if (__any_sync(0xffffffffu, big * zc > 1.0f)) {
 #pragma unroll
     for (int i = 0; i < 32; i++) {
