@@ -449,29 +449,13 @@ def vedizen_ops(dev, batch, context, heads=32, width=4096, ff=14336, chunk=2048)
     pk = peaks()
     bf = lambda *s: torch.randn(*s, device=dev).to(torch.bfloat16)
     T, out = batch * context, {}
+    d, e, H = 64, 128, heads
+    n_mix = 2 * H * d + 2 * H * e + 16
 
     def put(name, us, bytes_=0, tensor=0, fp32=0):
         roof = max(bytes_ / (pk["hbm_gbs"] * 1e9), tensor / (pk["bf16_tflops"] * 1e12), fp32 / 72.6e12) * 1e6
         out[name] = {"us": round(us, 1), "roofline_us": round(roof, 1), "frac": round(roof / us, 3)}
 
-    # linears: into gated units and mixer columns, and from both into the residual stream
-    d, e = 64, 128
-    H = heads
-    n_mix = 2 * H * d + 2 * H * e + 16
-    for name, rows in (("prefill", T), ("decode", batch)):
-        h, res = bf(rows, width), torch.randn(rows, width, device=dev)
-        w_in, w_out = bf(n_mix + 2 * ff, width), bf(width, H * e + ff)
-        cat, norm = bf(rows, H * e + ff), (0.5, torch.ones(width, device=dev), torch.zeros(width, device=dev))
-        n = 10 if rows == T else 40
-        put(f"linear_in_{name}", _time_us(lambda: HL.linear_glu(h, w_in, None, n_mix, 7.0, cat[:, H * e:]), n),
-            2 * (w_in.numel() + h.numel() + rows * (n_mix + ff)), tensor=2 * rows * w_in.numel())
-        put(f"linear_in_{name}_plain", _time_us(lambda: HL.linear(h, w_in), n), 2 * (w_in.numel() + h.numel() + rows * w_in.shape[0]),
-            tensor=2 * rows * w_in.numel())
-        put(f"linear_out_{name}", _time_us(lambda: HL.linear_residual(cat, w_out, res, None, norm), n),
-            2 * (w_out.numel() + cat.numel()) + rows * width * 10, tensor=2 * rows * w_out.numel())
-        put(f"linear_out_{name}_plain", _time_us(lambda: HL.linear(cat, w_out, out_f32=True), n), 2 * (w_out.numel() + cat.numel()) + rows * width * 4,
-            tensor=2 * rows * w_out.numel())
-        del h, res, w_in, w_out, cat
     # the start of the stream (embedding, norm) beside the Llama's norm
     from tpp_pytorch_extension_b200._C import _fused_llm_infer as F
     table, norm = bf(32000, width), (0.5, torch.ones(width, device=dev), torch.zeros(width, device=dev))
@@ -531,6 +515,22 @@ def vedizen_ops(dev, batch, context, heads=32, width=4096, ff=14336, chunk=2048)
         q1 = bf(batch, G, 1, H // G, hd)
         put(f"llama_attn_decode_kv{G}", _time_us(lambda: A.attention(q1, k1, v1, None, context), 40), 2 * 2 * batch * G * context * hd)
         del k1, v1, q1
+    # linears: into gated units and mixer columns, and from both into the residual stream (last: they
+    # run at the power limit, which slows what follows)
+    for name, rows in (("prefill", T), ("decode", batch)):
+        h, res = bf(rows, width), torch.randn(rows, width, device=dev)
+        w_in, w_out = bf(n_mix + 2 * ff, width), bf(width, H * e + ff)
+        cat, norm = bf(rows, H * e + ff), (0.5, torch.ones(width, device=dev), torch.zeros(width, device=dev))
+        n = 10 if rows == T else 40
+        put(f"linear_in_{name}", _time_us(lambda: HL.linear_glu(h, w_in, None, n_mix, 7.0, cat[:, H * e:]), n),
+            2 * (w_in.numel() + h.numel() + rows * (n_mix + ff)), tensor=2 * rows * w_in.numel())
+        put(f"linear_in_{name}_plain", _time_us(lambda: HL.linear(h, w_in), n), 2 * (w_in.numel() + h.numel() + rows * w_in.shape[0]),
+            tensor=2 * rows * w_in.numel())
+        put(f"linear_out_{name}", _time_us(lambda: HL.linear_residual(cat, w_out, res, None, norm), n),
+            2 * (w_out.numel() + cat.numel()) + rows * width * 10, tensor=2 * rows * w_out.numel())
+        put(f"linear_out_{name}_plain", _time_us(lambda: HL.linear(cat, w_out, out_f32=True), n), 2 * (w_out.numel() + cat.numel()) + rows * width * 4,
+            tensor=2 * rows * w_out.numel())
+        del h, res, w_in, w_out, cat
     return out
 
 

@@ -202,6 +202,22 @@ def test_diff_attention_sizes(cuda, dtype, sizes):
         assert U.err(got.reshape(B * T, -1), want.reshape(B * T, -1)) < U.TOL[dtype], cut
 
 
+@pytest.mark.parametrize("dim,vdim,B,chunk", [(64, 128, 40, 700), (128, 128, 2, 610), (32, 40, 3, 2000)])
+def test_diff_attention_long_chunks(cuda, dim, vdim, B, chunk):
+    """Many tiles per query tile and many pages per warp, with enough sequences that one block takes a whole chunk; unequal
+    padding moves the chunks against the pages."""
+    cfg = U.config([U.attn(8, 4, dim, vdim, chunk, dim ** -0.5, 20.0, mlp=None)], width=64)
+    w = P.random_model(cfg, seed=3, gain=3.0)
+    T, start = 900, [(31 * b) % 170 for b in range(B)]
+    h = rnd(1, B, T, 64)
+    some = sorted({0, 1, B - 1})
+    want = plain_batch(lambda x: P.diff_attention(x, w, "l0.mix", cfg["layers"][0]["mixer"], cfg["norm"]["eps"]), h[some], [start[b] for b in some])
+    mix = mixer_of(cfg, w, 0, cuda, torch.bfloat16)
+    for cut in ([10 ** 6], [600, 299, 1], [869, 1]):
+        got = mixer_over(mix, h, cut, cuda, torch.bfloat16, start)[some]
+        assert U.err(got.reshape(-1, 64), want.reshape(-1, 64)) < U.TOL[torch.bfloat16], cut
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("softcap,gain", [(0.5, 3.0), (2.0, 3.0), (64.0, 3.0), (64.0, 30.0), (200.0, 3.0)])
 def test_scores_far_above_and_below_the_cap(cuda, dtype, softcap, gain):
